@@ -63,10 +63,11 @@ int omc_latent_kv_store(const float* dkv, long long ld, int T, int r, int dr, co
                         int rot_dims, const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages,
                         int page_size, void* pool, int pool_dt, void* stream);
 
-/* omc_latent_kv_store and omc_rotary_q in one launch; w, pool, q and qcat share the dtype dt. */
+/* omc_latent_kv_store and omc_rotary_q in one launch; w, pool and qcat share the dtype dt, q is of q_dt. dkv NULL: only the queries
+ * (a layer that attends to another layer's cached rows). qn != NULL (dtype dt): receives the unrotated query parts, [T][H * dn]. */
 int omc_latent_rope_store(const float* dkv, long long ld, int T, int r, int dr, const void* w, float eps, const float* cs, int rot_dims,
                           const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size, void* pool,
-                          const void* q, long long ldq, int H, int dn, void* qcat, int dt, void* stream);
+                          const void* q, int q_dt, long long ldq, int H, int dn, void* qcat, void* qn, int dt, void* stream);
 
 /* Rotated query parts: q [T, H * (dn + dr)] of in_dt (per head dn unrotated then dr rotated dims) -> qcat[t][h][r + j] for
  * j < dr (qcat is [T, H, r + dr] of q_dt; its first r columns per head are written by the absorbing omc_linear). */
@@ -75,16 +76,18 @@ int omc_rotary_q(const void* q, int in_dt, long long ldq, int T, int H, int dn, 
 
 /* Paged latent attention, any sizes (the plain kernel: fp32 arithmetic, one CTA per (row, head)).
  * qcat [T, H, r + dr] (absorbed query | rotated query), pool as omc_latent_kv_store writes it. Row t of slot[t] at position
- * pos[t] sees the cached entries 0..pos[t] of its slot: score_j = qcat[t,h] . entry_j * scale, softmax over j with the optional
- * extra denominator term exp(sink[h]) (sink fp32 [H] or NULL), out[t,h,:] = sum_j p_j entry_j[:r] (fp32 [T, H, r]). r <= 1024. */
+ * pos[t] sees the last min(pos[t] + 1, window) cached entries of its slot: score_j = qcat[t,h] . entry_j * scale, softmax over j with the optional
+ * extra denominator term exp(sink[h]) (sink fp32 [H] or NULL), out[t,h,:] = sum_j p_j entry_j[:r] (fp32 [T, H, r]), times
+ * sigmoid(gate[t * ldg + h]) with gate != NULL (fp32: one gate per row and head). r <= 1024. */
 int omc_latent_attn(const void* qcat, int q_dt, int T, int H, int r, int dr, const void* pool, int pool_dt,
                     const int32_t* block_table, int max_pages, int page_size, const int32_t* pos, const int32_t* slot,
-                    const float* sink, float scale, float* out, void* stream);
+                    const float* sink, int window, const float* gate, long long ldg, float scale, float* out, void* stream);
 
 /* Tensor-core version of the same (bf16 only; r a multiple of 16 up to 512, dr a multiple of 16, H <= 64): mma.sync over 64-key
  * tiles that serve as keys AND values; the 64 rows of a tile are (token, head) pairs. The host lists the work:
  *   items[i]  = int32[8] (first_row, n_tok, slot, first_pos, key_begin, key_end, part_slot, 0): n_tok <= 64 / H consecutive rows
- *               of one request at positions first_pos.. against the cached keys [key_begin, key_end) (clipped causally per row).
+ *               of one request at positions first_pos.. against the cached keys [key_begin, key_end) (clipped per row to what the
+ *               row sees: causally and by the window).
  *               part_slot < 0: the item sees all its keys and writes `out`; else it writes its (max, sum, unnormalised output)
  *               partial to ws_o[part_slot][64][r] / ws_ml[part_slot][64][2] (long decode contexts cut into key ranges);
  *   merges[i] = int32[4] (first_row * H, n_rows, first part_slot, n_parts): partials that belong together.
@@ -92,12 +95,12 @@ int omc_latent_attn(const void* qcat, int q_dt, int T, int H, int r, int dr, con
  * omc_latent_attn up to the bf16 rounding of the probabilities. */
 int omc_latent_attn_mma(const void* qcat, int T, int H, int r, int dr, const void* pool, const int32_t* block_table, int max_pages,
                         int page_size, const int32_t* items, int n_items, const int32_t* merges, int n_merges, const float* sink,
-                        float scale, void* out, int out_dt, float* ws_o, float* ws_ml, void* stream);
+                        int window, const float* gate, long long ldg, float scale, void* out, int out_dt, float* ws_o, float* ws_ml, void* stream);
 
 /* The work list of a decode-only step, written on the device from pos / slot (one row per request, `parts` <= 64 key ranges each):
  * items int32 [B * parts][8], merges int32 [B][4] (untouched when parts == 1). Lets a CUDA graph replay the step as contexts grow. */
-int omc_latent_decode_items(const int32_t* pos, const int32_t* slot, int B, int H, int parts, int32_t* items, int32_t* merges,
-                            void* stream);
+int omc_latent_decode_items(const int32_t* pos, const int32_t* slot, int B, int H, int parts, int window, int32_t* items,
+                            int32_t* merges, void* stream);
 
 /* Router with score correction and identity experts. z fp32 [T, ldz]: logits of E_tot = experts + identity outputs, and, when
  * has_gate, one more column: the shared expert's gate logit. s = softmax(z[:E_tot] + bias) (bias fp32 [E_tot] or NULL);
@@ -105,12 +108,14 @@ int omc_latent_decode_items(const int32_t* pos, const int32_t* slot, int B, int 
  * weights = s of the chosen -> w fp32 [T, top], as they are (renorm 0) or divided by their sum (renorm 1: the softmax over the
  * chosen logits alone); gate[t] = sigmoid(z[t, E_tot]); counts[e] += 1 for every chosen e < experts (identity experts - the
  * last E_tot - experts outputs - take no rows). score OMC_ROUTER_SIGMOID: s = sigmoid(z + bias), every output on its own, instead
- * of the softmax. E_tot <= 4096, top <= 32. */
+ * of the softmax. groups > 1 with keep < groups: the outputs form `groups` equal groups of neighbours, a group's score is the sum of
+ * its two largest s (its one s when it has one), and only outputs of the `keep` best groups (ties: lowest index) can be chosen.
+ * w_scale multiplies the weights. E_tot <= 4096, top <= 32. */
 #define OMC_ROUTER_SOFTMAX 0
 #define OMC_ROUTER_SIGMOID 1
 int omc_router_topk(const float* z, long long ldz, int T, int E_tot, int experts, int top, const float* correction,
-                    const float* bias, int renorm, int score, int has_gate, int32_t* ids, float* w, float* gate, int32_t* counts,
-                    void* stream);
+                    const float* bias, int renorm, int score, int groups, int keep, float w_scale, int has_gate, int32_t* ids,
+                    float* w, float* gate, int32_t* counts, void* stream);
 
 /* Expert-sorted layout. plan: seg_start[e] = first row of expert e's segment, segments padded to whole `tile`-row tiles;
  * tile_group[i] = expert of tile i or -1 (max_tiles entries are written); counts and cursor are left zeroed for the next call.
@@ -314,6 +319,25 @@ int omc_diff_attn_pair(const void* q, long long ldq, int T, int H, int G, int d,
  * with long portions. */
 int omc_map_rows(float* x, long long ldx, int rows, int cols, int op, const float* A_log, const float* bias, int group, float p_exp,
                  void* stream);
+
+/* Layer norm after the residual sum, the experts' combine included:
+ *   v = alpha * x[t] + y[t] + sum_{j < top} w[t, j] * ys[slot_of[t, j]]     (y / ys NULL: no such term; slot_of < 0: skipped)
+ *   o = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * nw + nb
+ * -> x_out[t] (fp32, may be x; NULL to skip) and xb[t] (of xb_dt; NULL to skip). x / y / ys fp32; nw, nb [C] of w_dt. */
+int omc_ln_residual(const float* x, long long ldx, float alpha, const float* y, long long ldy, const float* ys, long long ldys,
+                    const int32_t* slot_of, const float* w, int top, const void* nw, const void* nb, int w_dt, float eps, float* x_out,
+                    long long ldxo, void* xb, int xb_dt, long long ldxb, int rows, int C, void* stream);
+
+/* Real-gated linear recurrent unit. Per channel c of `width` one fp32 state (state[slot][width]), two gates from block-diagonal
+ * products whose raw outputs sit in g [T, 2 * width]: block b of `blocks` holds its n = width / blocks recurrence gates at columns
+ * 2 n b .. and its n input gates behind them; gb (fp32 [2 * width], the same order, or NULL) is added.
+ *   r = sigmoid(g_r), i = sigmoid(g_i);  log a = -decay_scale * r * softplus(lam[c]);  S <- a S + sqrt(1 - a^2) * i * u[t, c]
+ *   out[t, c] = S * gelu_tanh(y[t, c])      (y fp32 rows or NULL: out = S)
+ * The decay is applied as S + expm1(log a) S. u and out of dtype dt. Portions and the zero start at position 0 as in
+ * omc_linear_state_scan; rows: T, the number of rows over all portions (it selects how the tokens are spread over warps). */
+int omc_rglru_scan(const void* u, int dt, long long ldu, const float* g, long long ldg, const float* gb, const float* lam, const float* y,
+                   long long ldy, float* state, void* out, long long ldo, const int32_t* row_begin, int portions, const int32_t* pos,
+                   const int32_t* slot, int rows, int width, int blocks, float decay_scale, void* stream);
 
 #ifdef __cplusplus
 }

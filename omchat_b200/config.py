@@ -176,7 +176,9 @@ class RotarySpec:
 class LatentAttentionSpec:
     """Attention whose keys and values are up-projections of a cached latent of width kv_rank plus one rotated key part of
     width rot_dim shared by the heads. q_rank: queries go through a normed latent of that width (None: one projection).
-    sink: the softmax denominator has one more learned term per head."""
+    sink: the softmax denominator has one more learned term per head. window: keys a row sees behind itself, itself included
+    (None: all). head_gate: every head's output is multiplied by a sigmoid of a projection of the mixer's input. kv_from: the
+    layer whose cached rows this one attends to (it projects no keys or values of its own and caches nothing)."""
     heads: int
     dim: int        # unrotated query / key dimensions per head
     rot_dim: int    # rotated query / key dimensions per head
@@ -186,6 +188,9 @@ class LatentAttentionSpec:
     rot: RotarySpec = None
     q_rank: Optional[int] = None
     sink: bool = False
+    window: Optional[int] = None
+    head_gate: bool = False
+    kv_from: Optional[int] = None
 
 
 @dataclass
@@ -716,3 +721,137 @@ class VefunexConfig:
         return {"architecture": "Vefunex", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps},
                 "residual_mult": self.residual_mult, "logit_softcap": self.logit_softcap, "canon": {"taps": self.canon_taps}, "layers": out,
                 "kv_page_size": self.kv_page_size, "eos_token_id": self.eos_token_id, "pad_token_id": self.pad_token_id}
+
+
+# --------------------------------------------------------------------------------------------------------------------- Munevik
+@dataclass
+class GatedLruSpec:
+    """Gated linear recurrent unit: `width` channels with one fp32 state each; an input branch behind a causal convolution of `conv`
+    taps (with bias, no activation) whose recurrence and input gates are block-diagonal projections of `blocks` square matrices,
+    and a gelu branch that multiplies the states. S <- a S + sqrt(1 - a^2) i u with a = exp(-decay_scale r softplus(lam))."""
+    width: int
+    blocks: int
+    conv: int
+    decay_scale: float = 8.0
+
+
+@dataclass
+class ClampedMlpSpec:
+    """g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit), W_down (g sigmoid(1.702 g) (u + 1)), no biases."""
+    ff: int
+    limit: float
+
+
+@dataclass
+class GroupedMoeSpec:
+    """`experts` gated silu experts (no biases) of width expert_ff, `top` per token by the largest sigmoid router scores, weights
+    score * scale. groups / keep: experts form that many equal groups of neighbours, a group is scored by the sum of its two
+    largest scores, and only experts of the best `keep` groups can be chosen (1 / 1: no groups). shared_ff: width of an expert of
+    the same form that every token passes and that is added as it is (None: none)."""
+    experts: int
+    top: int
+    expert_ff: int
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared_ff: Optional[int] = None
+
+
+@dataclass
+class MunevikLayerSpec:
+    type: str                      # 'latent_attention' | 'rglru'
+    mixer: object                  # LatentAttentionSpec | GatedLruSpec
+    mlp: object                    # ClampedMlpSpec | GroupedMoeSpec | None
+
+
+@dataclass
+class MunevikConfig:
+    model_type: str = "munevik"
+    vocab_size: int = 0
+    hidden_size: int = 0
+    norm_eps: float = 1e-6
+    postln_alpha: float = 1.0      # a sublayer's residual: x <- norm(postln_alpha * x + sublayer(x))
+    layers: List[MunevikLayerSpec] = field(default_factory=list)
+    kv_page_size: int = 64         # engine knob: tokens per cache page
+    eos_token_id: int = -1
+    pad_token_id: int = 0
+
+    MIXERS = ("latent_attention", "rglru")
+    SWISH_SLOPE = 1.702            # the dense feed-forward's gate is g * sigmoid(SWISH_SLOPE * g)
+    UP_SHIFT = 1.0                 # ... times (u + UP_SHIFT)
+
+    @staticmethod
+    def _latent(m: dict, i: int, layers: list) -> LatentAttentionSpec:
+        rot, mask, src = m.get("rot") or {}, m.get("mask") or {}, m.get("kv_from")
+        rspec = RotarySpec(dims=int(rot.get("dims", m["rot_dim"])), base=float(rot.get("base", 10000.0)))
+        spec = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                                   scale=float(m["scale"]), rot=rspec, window=int(mask["size"]) if mask.get("size") is not None else None,
+                                   head_gate=True, kv_from=int(src) if src is not None else None)
+        if min(spec.heads, spec.dim, spec.vdim, spec.kv_rank) < 1 or spec.rot_dim < 0 or rspec.dims % 2 or not 0 <= rspec.dims <= spec.rot_dim or \
+                (spec.window is not None and spec.window < 1):
+            raise ValueError(f"layer {i}: inconsistent attention sizes")
+        if spec.kv_from is not None:
+            s = layers[spec.kv_from].mixer if 0 <= spec.kv_from < i else None
+            if not isinstance(s, LatentAttentionSpec) or s.kv_from is not None:
+                raise ValueError(f"layer {i}: kv_from must name an earlier latent-attention layer with a cache of its own")
+            if (s.kv_rank, s.rot_dim, s.rot) != (spec.kv_rank, spec.rot_dim, spec.rot):
+                raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation must be those of layer {spec.kv_from}")
+        return spec
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "MunevikConfig":
+        layers = []
+        for i, ld in enumerate(d["layers"]):
+            typ, m = ld["type"], ld["mixer"]
+            if typ == "latent_attention":
+                mix = cls._latent(m, i, layers)
+            elif typ == "rglru":
+                mix = GatedLruSpec(width=int(m["width"]), blocks=int(m["blocks"]), conv=int(m["conv"]))
+                if min(mix.width, mix.blocks, mix.conv) < 1 or mix.width % mix.blocks:
+                    raise ValueError(f"layer {i}: inconsistent recurrence sizes")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {typ!r}")
+            md, mlp = ld.get("mlp"), None
+            if md:
+                kind = md.get("kind", "dense")
+                if kind == "dense":
+                    mlp = ClampedMlpSpec(ff=int(md["ff"]), limit=float(md["limit"]))
+                elif kind == "moe":
+                    r, g, sh = md["router"], md["router"].get("groups") or {}, md.get("shared")
+                    mlp = GroupedMoeSpec(experts=int(r["experts"]), top=int(r["top"]), expert_ff=int(md["expert"]["ff"]), groups=int(g.get("count", 1)),
+                                         keep=int(g.get("keep", g.get("count", 1))), scale=float(r.get("scale", 1.0)),
+                                         shared_ff=int(sh["ff"]) if sh else None)
+                    if min(mlp.experts, mlp.top, mlp.expert_ff, mlp.groups) < 1 or mlp.experts % mlp.groups or not 1 <= mlp.keep <= mlp.groups:
+                        raise ValueError(f"layer {i}: inconsistent expert sizes")
+                    if mlp.top > mlp.keep * (mlp.experts // mlp.groups):
+                        raise ValueError(f"layer {i}: fewer experts can be chosen than a token uses")
+                else:
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
+            layers.append(MunevikLayerSpec(type=typ, mixer=mix, mlp=mlp))
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)),
+                   postln_alpha=float(d.get("postln_alpha", 1.0)), layers=layers, kv_page_size=int(d.get("kv_page_size", 64)),
+                   eos_token_id=int(d.get("eos_token_id", -1)), pad_token_id=int(d.get("pad_token_id", 0)))
+
+    def to_dict(self) -> dict:
+        """The config.json form (round-trips through from_dict)."""
+        out = []
+        for l in self.layers:
+            m, s, mlp = l.mixer, l.mlp, None
+            if isinstance(m, LatentAttentionSpec):
+                md = {"dim": m.dim, "heads": m.heads, "kv_rank": m.kv_rank, "rot": {"base": m.rot.base, "dims": m.rot.dims}, "rot_dim": m.rot_dim,
+                      "scale": m.scale, "vdim": m.vdim}
+                if m.window is not None:
+                    md["mask"] = {"size": m.window}
+                if m.kv_from is not None:
+                    md["kv_from"] = m.kv_from
+            else:
+                md = {"blocks": m.blocks, "conv": m.conv, "width": m.width}
+            if isinstance(s, ClampedMlpSpec):
+                mlp = {"ff": s.ff, "kind": "dense", "limit": s.limit}
+            elif isinstance(s, GroupedMoeSpec):
+                mlp = {"expert": {"ff": s.expert_ff}, "kind": "moe", "shared": {"ff": s.shared_ff} if s.shared_ff else None,
+                       "router": {"experts": s.experts, "groups": {"count": s.groups, "keep": s.keep}, "scale": s.scale, "top": s.top}}
+            out.append({"type": l.type, "mixer": md, "mlp": mlp})
+        return {"architecture": "Munevik", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps},
+                "postln_alpha": self.postln_alpha, "layers": out, "kv_page_size": self.kv_page_size, "eos_token_id": self.eos_token_id,
+                "pad_token_id": self.pad_token_id}

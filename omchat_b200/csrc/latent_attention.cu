@@ -64,38 +64,42 @@ __global__ void __launch_bounds__(128) rotary_q_kernel(const TI* __restrict__ q3
 }
 
 // Both of the above for one row in one launch (a step's decode rows pay per launch, not per byte): the cache append of the row's
-// latent and rotated key part, then the rotated query parts of all heads. All stored operands share one type.
-template <typename T>
+// latent and rotated key part (dkv NULL: the layer attends to another layer's rows and appends nothing), then the rotated query
+// parts of all heads, and with qn != NULL the unrotated query parts as rows of their own [T][H * dn] - for queries that arrive in
+// fp32 from a product they share with other outputs and leave as matrix operands of the storage type.
+template <typename T, typename TQ>
 __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __restrict__ dkv, long long ld, int r, int dr,
                                                                 const T* __restrict__ w, float eps, const float* __restrict__ cs,
                                                                 int rot_dims, const int32_t* __restrict__ pos,
                                                                 const int32_t* __restrict__ slot,
                                                                 const int32_t* __restrict__ block_table, int max_pages, int page_size,
-                                                                T* __restrict__ pool, const T* __restrict__ q, long long ldq, int H, int dn,
-                                                                T* __restrict__ qcat) {
+                                                                T* __restrict__ pool, const TQ* __restrict__ q, long long ldq, int H, int dn,
+                                                                T* __restrict__ qcat, T* __restrict__ qn) {
   __shared__ float red[33];
   const int t = blockIdx.x;
-  const float* row = dkv + (long long)t * ld;
   const int p = pos[t];
-  const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
-  T* dst = pool + ((long long)page * page_size + p % page_size) * (r + dr);
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < r; c += blockDim.x) ss = fmaf(row[c], row[c], ss);
-  ss = block_sum(ss, red);
-  const float rstd = 1.f / sqrtf(ss / (float)r + eps);
-  for (int c = threadIdx.x; c < r; c += blockDim.x) stf(dst + c, row[c] * rstd * ldf(w + c));
   const int half = rot_dims >> 1;
   const float* csr = cs + (long long)p * rot_dims;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const float u = row[r + 2 * i], v = row[r + 2 * i + 1], co = csr[2 * i], si = csr[2 * i + 1];
-    stf(dst + r + 2 * i, u * co - v * si);
-    stf(dst + r + 2 * i + 1, v * co + u * si);
+  if (dkv != nullptr) {
+    const float* row = dkv + (long long)t * ld;
+    const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
+    T* dst = pool + ((long long)page * page_size + p % page_size) * (r + dr);
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < r; c += blockDim.x) ss = fmaf(row[c], row[c], ss);
+    ss = block_sum(ss, red);
+    const float rstd = 1.f / sqrtf(ss / (float)r + eps);
+    for (int c = threadIdx.x; c < r; c += blockDim.x) stf(dst + c, row[c] * rstd * ldf(w + c));
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      const float u = row[r + 2 * i], v = row[r + 2 * i + 1], co = csr[2 * i], si = csr[2 * i + 1];
+      stf(dst + r + 2 * i, u * co - v * si);
+      stf(dst + r + 2 * i + 1, v * co + u * si);
+    }
+    for (int c = rot_dims + threadIdx.x; c < dr; c += blockDim.x) stf(dst + r + c, row[r + c]);
   }
-  for (int c = rot_dims + threadIdx.x; c < dr; c += blockDim.x) stf(dst + r + c, row[r + c]);
   // queries: every (head, pair) is one unit of work
   for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
     const int h = i / half, j = i - h * half;
-    const T* src = q + (long long)t * ldq + (long long)h * (dn + dr) + dn;
+    const TQ* src = q + (long long)t * ldq + (long long)h * (dn + dr) + dn;
     T* qd = qcat + ((long long)t * H + h) * (r + dr) + r;
     const float u = ldf(src + 2 * j), v = ldf(src + 2 * j + 1), co = csr[2 * j], si = csr[2 * j + 1];
     stf(qd + 2 * j, u * co - v * si);
@@ -106,6 +110,16 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
     const int h = i / rest, c = rot_dims + (i - h * rest);
     stf(qcat + ((long long)t * H + h) * (r + dr) + r + c, ldf(q + (long long)t * ldq + (long long)h * (dn + dr) + dn + c));
   }
+  if (qn != nullptr) {
+    for (int i = threadIdx.x; i < H * dn; i += blockDim.x) {
+      const int h = i / dn, c = i - h * dn;
+      stf(qn + (long long)t * H * dn + i, ldf(q + (long long)t * ldq + (long long)h * (dn + dr) + c));
+    }
+  }
+}
+
+__device__ __forceinline__ float head_gate_f(const float* gate, long long ldg, long long t, int h) {
+  return gate != nullptr ? 1.f / (1.f + expf(-gate[t * ldg + h])) : 1.f;
 }
 
 constexpr int kLatWarps = 4;
@@ -120,7 +134,8 @@ __global__ void __launch_bounds__(kLatWarps * 32) latent_attn_kernel(const TQ* _
                                                                      const int32_t* __restrict__ block_table, int max_pages,
                                                                      int page_size, const int32_t* __restrict__ pos,
                                                                      const int32_t* __restrict__ slot,
-                                                                     const float* __restrict__ sink, float scale,
+                                                                     const float* __restrict__ sink, int window,
+                                                                     const float* __restrict__ gate, long long ldg, float scale,
                                                                      float* __restrict__ out) {
   extern __shared__ float sm[];  // q [r + dr] | acc [kLatWarps][r] | m [kLatWarps] | l [kLatWarps]
   const int t = blockIdx.x, h = blockIdx.y;
@@ -139,7 +154,7 @@ __global__ void __launch_bounds__(kLatWarps * 32) latent_attn_kernel(const TQ* _
   float acc[kLatMaxPerLane];
 #pragma unroll
   for (int i = 0; i < kLatMaxPerLane; ++i) acc[i] = 0.f;
-  for (int j = warp; j < n_keys; j += kLatWarps) {
+  for (int j = max(0, n_keys - window) + warp; j < n_keys; j += kLatWarps) {
     const TC* kr = pool + ((long long)bt[j / page_size] * page_size + j % page_size) * D;
     float d = 0.f;
     for (int c = lane; c < D; c += 32) d = fmaf(sq[c], ldf(kr + c), d);
@@ -175,7 +190,7 @@ __global__ void __launch_bounds__(kLatWarps * 32) latent_attn_kernel(const TQ* _
     f[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - mt);
     lt += s_l[w] * f[w];
   }
-  const float inv = 1.f / lt;
+  const float inv = head_gate_f(gate, ldg, t, h) / lt;
   float* o = out + ((long long)t * H + h) * r;
   for (int c = threadIdx.x; c < r; c += blockDim.x) {
     float v = 0.f;
@@ -206,19 +221,19 @@ extern "C" int omc_latent_kv_store(const float* dkv, long long ld, int T, int r,
 
 extern "C" int omc_latent_rope_store(const float* dkv, long long ld, int T, int r, int dr, const void* w, float eps, const float* cs,
                                      int rot_dims, const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages,
-                                     int page_size, void* pool, const void* q, long long ldq, int H, int dn, void* qcat, int dt,
-                                     void* stream) {
-  if (dkv == nullptr || w == nullptr || cs == nullptr || pos == nullptr || slot == nullptr || block_table == nullptr || pool == nullptr ||
-      q == nullptr || qcat == nullptr || T < 0 || r <= 0 || dr < 0 || rot_dims < 0 || rot_dims > dr || (rot_dims & 1) || page_size <= 0 ||
-      max_pages <= 0 || H <= 0 || dn < 0)
+                                     int page_size, void* pool, const void* q, int q_dt, long long ldq, int H, int dn, void* qcat, void* qn,
+                                     int dt, void* stream) {
+  if (cs == nullptr || pos == nullptr || q == nullptr || qcat == nullptr || T < 0 || r <= 0 || dr < 0 || rot_dims < 0 || rot_dims > dr ||
+      (rot_dims & 1) || H <= 0 || dn < 0 ||
+      (dkv != nullptr && (w == nullptr || slot == nullptr || block_table == nullptr || pool == nullptr || page_size <= 0 || max_pages <= 0)))
     return set_error(OMC_ERR_ARG, "omc_latent_rope_store: bad argument");
   if (T == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  OMC_DT_SWITCH(dt, TT, {
-    latent_rope_store_kernel<TT><<<T, 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, pos, slot, block_table,
-                                                    max_pages, page_size, static_cast<TT*>(pool), static_cast<const TT*>(q), ldq, H, dn,
-                                                    static_cast<TT*>(qcat));
-  })
+  OMC_DT_SWITCH(dt, TT, OMC_DT_SWITCH(q_dt, TQ, {
+    latent_rope_store_kernel<TT, TQ><<<T, 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, pos, slot, block_table,
+                                                        max_pages, page_size, static_cast<TT*>(pool), static_cast<const TQ*>(q), ldq, H, dn,
+                                                        static_cast<TT*>(qcat), static_cast<TT*>(qn));
+  }))
   return check_launch("omc_latent_rope_store");
 }
 
@@ -237,7 +252,8 @@ extern "C" int omc_rotary_q(const void* q32, int in_dt, long long ldq, int T, in
 
 extern "C" int omc_latent_attn(const void* qcat, int q_dt, int T, int H, int r, int dr, const void* pool, int pool_dt,
                                const int32_t* block_table, int max_pages, int page_size, const int32_t* pos, const int32_t* slot,
-                               const float* sink, float scale, float* out, void* stream) {
+                               const float* sink, int window, const float* gate, long long ldg, float scale, float* out, void* stream) {
+  if (window < 1) return set_error(OMC_ERR_ARG, "omc_latent_attn: the window holds at least the row itself");
   if (qcat == nullptr || pool == nullptr || block_table == nullptr || pos == nullptr || slot == nullptr || out == nullptr || T < 0 ||
       H <= 0 || r <= 0 || dr < 0 || page_size <= 0 || max_pages <= 0)
     return set_error(OMC_ERR_ARG, "omc_latent_attn: bad argument");
@@ -249,7 +265,7 @@ extern "C" int omc_latent_attn(const void* qcat, int q_dt, int T, int H, int r, 
   OMC_DT_SWITCH(q_dt, TQ, OMC_DT_SWITCH(pool_dt, TC, {
     latent_attn_kernel<TQ, TC><<<dim3(T, H), kLatWarps * 32, smem, st>>>(static_cast<const TQ*>(qcat), H, r, dr,
                                                                          static_cast<const TC*>(pool), block_table, max_pages,
-                                                                         page_size, pos, slot, sink, scale, out);
+                                                                         page_size, pos, slot, sink, window, gate, ldg, scale, out);
   }))
   return check_launch("omc_latent_attn");
 }
@@ -304,6 +320,9 @@ struct LatMmaArgs {
   void* out;     // [T * H][r] fp32 or bf16
   float* ws_o;   // [part_slot][64][r]
   float* ws_ml;  // [part_slot][64][2]
+  const float* gate;  // [T][ldg] fp32 or NULL: head h's output is multiplied by sigmoid(gate[t][h])
+  long long ldg;
+  int window;         // row i sees the keys j <= i with i - j < window
   int max_pages, page_size, H, r, dr;
   float scale_log2;
   int two_buffers;  // shared memory holds two key tiles
@@ -339,6 +358,7 @@ __global__ void __launch_bounds__(128 * VS) latent_attn_mma_kernel(LatMmaArgs a)
   // last key (inclusive) each of this thread's two rows may see
   const int lim0 = row0 < n_rows ? first_pos + row0 / a.H : -1;
   const int lim1 = row1 < n_rows ? first_pos + row1 / a.H : -1;
+  const int low0 = lim0 - a.window + 1, low1 = lim1 - a.window + 1;  // first keys they see
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   float o[NV][4];
 #pragma unroll
@@ -423,10 +443,10 @@ __global__ void __launch_bounds__(128 * VS) latent_attn_mma_kernel(LatMmaArgs a)
 #pragma unroll
     for (int n = 0; n < NS; ++n) {
       const int key = j0 + kofs + n * 8 + 2 * t4;
-      s[n][0] = key <= lim0 ? s[n][0] * a.scale_log2 : -INFINITY;
-      s[n][1] = key + 1 <= lim0 ? s[n][1] * a.scale_log2 : -INFINITY;
-      s[n][2] = key <= lim1 ? s[n][2] * a.scale_log2 : -INFINITY;
-      s[n][3] = key + 1 <= lim1 ? s[n][3] * a.scale_log2 : -INFINITY;
+      s[n][0] = (key <= lim0 && key >= low0) ? s[n][0] * a.scale_log2 : -INFINITY;
+      s[n][1] = (key + 1 <= lim0 && key + 1 >= low0) ? s[n][1] * a.scale_log2 : -INFINITY;
+      s[n][2] = (key <= lim1 && key >= low1) ? s[n][2] * a.scale_log2 : -INFINITY;
+      s[n][3] = (key + 1 <= lim1 && key + 1 >= low1) ? s[n][3] * a.scale_log2 : -INFINITY;
       mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
       mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
     }
@@ -531,7 +551,11 @@ __global__ void __launch_bounds__(128 * VS) latent_attn_mma_kernel(LatMmaArgs a)
       if (row0 < n_rows) d0 += exp2f(a.sink[row0 % a.H] * 1.4426950408889634f - m0);
       if (row1 < n_rows) d1 += exp2f(a.sink[row1 % a.H] * 1.4426950408889634f - m1);
     }
-    const float i0 = 1.f / d0, i1 = 1.f / d1;
+    float i0 = 1.f / d0, i1 = 1.f / d1;
+    if (a.gate != nullptr) {
+      if (row0 < n_rows) i0 *= head_gate_f(a.gate, a.ldg, first_row + row0 / a.H, row0 % a.H);
+      if (row1 < n_rows) i1 *= head_gate_f(a.gate, a.ldg, first_row + row1 / a.H, row1 % a.H);
+    }
     TO* out0 = static_cast<TO*>(a.out) + ((long long)first_row * a.H + row0) * a.r;
     TO* out1 = static_cast<TO*>(a.out) + ((long long)first_row * a.H + row1) * a.r;
 #pragma unroll
@@ -569,8 +593,9 @@ __global__ void __launch_bounds__(128 * VS) latent_attn_mma_kernel(LatMmaArgs a)
 constexpr int kMergeMaxParts = 64;
 template <typename TO>
 __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const int32_t* __restrict__ merges, const float* __restrict__ ws_o,
-                                                                const float* __restrict__ ws_ml, const float* __restrict__ sink, int H,
-                                                                int r, TO* __restrict__ out) {
+                                                                const float* __restrict__ ws_ml, const float* __restrict__ sink,
+                                                                const float* __restrict__ gate, long long ldg, int H, int r,
+                                                                TO* __restrict__ out) {
   __shared__ float s_f[kMergeMaxParts];
   __shared__ float s_inv;
   const int32_t* mg = merges + blockIdx.x * 4;
@@ -593,7 +618,7 @@ __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const int32_t* _
     }
     den = seq_warp_sum(den);
     if (sink != nullptr) den += exp2f(sk - mt);
-    if (lane == 0) s_inv = 1.f / den;
+    if (lane == 0) s_inv = head_gate_f(gate, ldg, (qrow0 + row) / H, (qrow0 + row) % H) / den;
   }
   __syncthreads();
   const float inv = s_inv;
@@ -615,22 +640,22 @@ __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const int32_t* _
 }
 
 // Work list of a decode-only step written on the device (so that the step can be replayed from a CUDA graph while the contexts
-// grow): row b at position pos[b] sees pos[b] + 1 keys, cut into `parts` ranges of whole 64-key tiles (ranges past the end stay
+// grow): row b at position pos[b] sees the last min(pos[b] + 1, window) keys, cut into `parts` ranges of whole 64-key tiles (ranges past the end stay
 // empty and contribute nothing to the merge).
-__global__ void latent_decode_items_kernel(const int32_t* __restrict__ pos, const int32_t* __restrict__ slot, int B, int H, int parts,
+__global__ void latent_decode_items_kernel(const int32_t* __restrict__ pos, const int32_t* __restrict__ slot, int B, int H, int parts, int window,
                                            int32_t* __restrict__ items, int32_t* __restrict__ merges) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= B * parts) return;
   const int b = i / parts, j = i - b * parts;
-  const int keys = pos[b] + 1;
-  const int span = ((keys + parts - 1) / parts + kMmaKeys - 1) / kMmaKeys * kMmaKeys;
+  const int keys = pos[b] + 1, low = max(0, keys - window);
+  const int span = ((keys - low + parts - 1) / parts + kMmaKeys - 1) / kMmaKeys * kMmaKeys;
   int32_t* it = items + (long long)i * 8;
   it[0] = b;
   it[1] = 1;
   it[2] = slot[b];
   it[3] = pos[b];
-  it[4] = min(j * span, keys);
-  it[5] = min((j + 1) * span, keys);
+  it[4] = min(low + j * span, keys);
+  it[5] = min(low + (j + 1) * span, keys);
   it[6] = parts > 1 ? i : -1;
   it[7] = 0;
   if (j == 0 && parts > 1) {
@@ -665,8 +690,9 @@ static int launch_lat_mma(const LatMmaArgs& a, int out_dt, int n_items, size_t s
 
 extern "C" int omc_latent_attn_mma(const void* qcat, int T, int H, int r, int dr, const void* pool, const int32_t* block_table,
                                    int max_pages, int page_size, const int32_t* items, int n_items, const int32_t* merges,
-                                   int n_merges, const float* sink, float scale, void* out, int out_dt, float* ws_o, float* ws_ml,
-                                   void* stream) {
+                                   int n_merges, const float* sink, int window, const float* gate, long long ldg, float scale, void* out,
+                                   int out_dt, float* ws_o, float* ws_ml, void* stream) {
+  if (window < 1) return set_error(OMC_ERR_ARG, "omc_latent_attn_mma: the window holds at least the row itself");
   if (qcat == nullptr || pool == nullptr || block_table == nullptr || items == nullptr || out == nullptr || T < 0 || H <= 0 ||
       page_size <= 0 || max_pages <= 0 || n_items < 0 || n_merges < 0 || (n_merges > 0 && (merges == nullptr || ws_o == nullptr || ws_ml == nullptr)))
     return set_error(OMC_ERR_ARG, "omc_latent_attn_mma: bad argument");
@@ -682,7 +708,7 @@ extern "C" int omc_latent_attn_mma(const void* qcat, int T, int H, int r, int dr
     smem = (size_t)(kMmaRows + kMmaKeys) * (D + 8) * sizeof(bf16_t) + extra;
   }
   if (smem > 227 * 1024) return set_error(OMC_ERR_SHAPE, "omc_latent_attn_mma: rows too wide for shared memory");
-  LatMmaArgs a{static_cast<const bf16_t*>(qcat), static_cast<const bf16_t*>(pool), block_table, items, sink, out, ws_o, ws_ml,
+  LatMmaArgs a{static_cast<const bf16_t*>(qcat), static_cast<const bf16_t*>(pool), block_table, items, sink, out, ws_o, ws_ml, gate, ldg, window,
                max_pages, page_size, H, r, dr, scale * 1.4426950408889634f, two};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int rc;
@@ -693,19 +719,19 @@ extern "C" int omc_latent_attn_mma(const void* qcat, int T, int H, int r, int dr
   else rc = launch_lat_mma<4, 16>(a, out_dt, n_items, smem, st);  // 16 warps: four per row group, 128 value columns and 16 keys each
   if (rc != OMC_OK || n_merges == 0) return rc;
   if (out_dt == OMC_DT_BF16)
-    latent_attn_merge_kernel<bf16_t><<<dim3(n_merges, kMmaRows), 128, 0, st>>>(merges, ws_o, ws_ml, sink, H, r, static_cast<bf16_t*>(out));
+    latent_attn_merge_kernel<bf16_t><<<dim3(n_merges, kMmaRows), 128, 0, st>>>(merges, ws_o, ws_ml, sink, gate, ldg, H, r, static_cast<bf16_t*>(out));
   else
-    latent_attn_merge_kernel<float><<<dim3(n_merges, kMmaRows), 128, 0, st>>>(merges, ws_o, ws_ml, sink, H, r, static_cast<float*>(out));
+    latent_attn_merge_kernel<float><<<dim3(n_merges, kMmaRows), 128, 0, st>>>(merges, ws_o, ws_ml, sink, gate, ldg, H, r, static_cast<float*>(out));
   return check_launch("omc_latent_attn_merge");
 }
 
-extern "C" int omc_latent_decode_items(const int32_t* pos, const int32_t* slot, int B, int H, int parts, int32_t* items, int32_t* merges,
-                                       void* stream) {
-  if (pos == nullptr || slot == nullptr || items == nullptr || B < 0 || H <= 0 || parts <= 0 || parts > kMergeMaxParts ||
+extern "C" int omc_latent_decode_items(const int32_t* pos, const int32_t* slot, int B, int H, int parts, int window, int32_t* items,
+                                       int32_t* merges, void* stream) {
+  if (pos == nullptr || slot == nullptr || items == nullptr || B < 0 || H <= 0 || parts <= 0 || parts > kMergeMaxParts || window < 1 ||
       (parts > 1 && merges == nullptr))
     return set_error(OMC_ERR_ARG, "omc_latent_decode_items: bad argument");
   if (B == 0) return OMC_OK;
   const int n = B * parts;
-  latent_decode_items_kernel<<<(n + 127) / 128, 128, 0, static_cast<cudaStream_t>(stream)>>>(pos, slot, B, H, parts, items, merges);
+  latent_decode_items_kernel<<<(n + 127) / 128, 128, 0, static_cast<cudaStream_t>(stream)>>>(pos, slot, B, H, parts, window, items, merges);
   return check_launch("omc_latent_decode_items");
 }

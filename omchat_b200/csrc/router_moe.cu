@@ -3,7 +3,9 @@
 //
 //   router:   s = softmax(z + bias) over ALL router outputs (experts, then identity experts); the choice is made on s + correction, the
 //             mixing weights are the uncorrected s of the chosen outputs - as they are, or divided by their sum (`renorm`), which is
-//             the softmax over the chosen logits alone. An identity expert returns its input,
+//             the softmax over the chosen logits alone; with a sigmoid score every output is scored on its own. Groups: outputs form
+//             equal groups of neighbours, a group's score is the sum of its two largest scores s, and only outputs of the best `keep`
+//             groups can be chosen. A factor may scale the weights. An identity expert returns its input,
 //             has no weights and takes no rows in the sorted layout. The shared expert's gate logit rides as one more column of z.
 //   plan:     one CTA: segment starts padded to whole row tiles, tile -> expert table, counters reset for the next call.
 //   scatter:  one CTA per row: the row is copied to a place in the segment of each chosen expert (atomic cursor per expert; the
@@ -17,18 +19,19 @@ namespace omc {
 
 constexpr int kRouteWarps = 4;
 
-// One warp per row. Shared memory per warp: s[E_tot] (softmax scores) and ch[E_tot] (choice values, -inf once taken).
+// One warp per row. Shared memory per warp: s[E_tot] (scores), ch[E_tot] (choice values, -inf once taken) and gs[groups] (group scores).
 __global__ void __launch_bounds__(kRouteWarps * 32) router_topk_kernel(const float* __restrict__ z, long long ldz, int T, int E_tot,
                                                                        int experts, int top, const float* __restrict__ correction,
-                                                                       const float* __restrict__ bias, int renorm, int score,
-                                                                       int has_gate, int32_t* __restrict__ ids, float* __restrict__ w,
+                                                                       const float* __restrict__ bias, int renorm, int score, int groups,
+                                                                       int keep, float w_scale, int has_gate, int32_t* __restrict__ ids, float* __restrict__ w,
                                                                        float* __restrict__ gate, int32_t* __restrict__ counts) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouteWarps + warp;
   if (t >= T) return;
-  float* s = sm + (size_t)warp * 2 * E_tot;
+  float* s = sm + (size_t)warp * (2 * E_tot + groups);
   float* ch = s + E_tot;
+  float* gs = ch + E_tot;
   const float* zr = z + (long long)t * ldz;
   float mx = -INFINITY;
   for (int e = lane; e < E_tot; e += 32) {
@@ -59,6 +62,27 @@ __global__ void __launch_bounds__(kRouteWarps * 32) router_topk_kernel(const flo
     }
   }
   __syncwarp();
+  if (keep < groups) {   // outputs outside the best groups cannot be chosen
+    const int n = E_tot / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+      for (int e = g * n; e < (g + 1) * n; ++e) {
+        const float v = s[e];
+        b2 = fmaxf(b2, fminf(b1, v));
+        b1 = fmaxf(b1, v);
+      }
+      gs[g] = n > 1 ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    // a group stays when fewer than `keep` others beat it (ties: the lower index wins); NaN scores keep every group
+    for (int g = lane; g < groups; g += 32) {
+      int better = 0;
+      for (int o = 0; o < groups; ++o) better += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
+      if (better >= keep)
+        for (int e = g * n; e < (g + 1) * n; ++e) ch[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
   for (int k = 0; k < top; ++k) {
     float bv = -INFINITY;
     int be = 0x7fffffff;
@@ -81,7 +105,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) router_topk_kernel(const flo
     if (be >= E_tot) be = k % E_tot;  // only with NaN logits: stay inside the tables
     if (lane == 0) {
       ids[(long long)t * top + k] = be;
-      w[(long long)t * top + k] = s[be];
+      w[(long long)t * top + k] = s[be] * w_scale;
       if (be < experts) atomicAdd(counts + be, 1);
       ch[be] = -INFINITY;
     }
@@ -90,7 +114,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) router_topk_kernel(const flo
   if (renorm && lane == 0) {   // softmax over the chosen alone: exp(z - max) / sum over the chosen, the common factor cancels
     float tot = 0.f;
     for (int k = 0; k < top; ++k) tot += w[(long long)t * top + k];
-    const float r = 1.f / tot;
+    const float r = w_scale / tot;
     for (int k = 0; k < top; ++k) w[(long long)t * top + k] *= r;
   }
   if (has_gate && lane == 0) gate[t] = 1.f / (1.f + expf(-zr[E_tot]));
@@ -293,21 +317,23 @@ __global__ void __launch_bounds__(256) moe_combine_depth_kernel(const float* __r
 using namespace omc;
 
 extern "C" int omc_router_topk(const float* z, long long ldz, int T, int E_tot, int experts, int top, const float* correction,
-                               const float* bias, int renorm, int score, int has_gate, int32_t* ids, float* w, float* gate, int32_t* counts,
-                               void* stream) {
+                               const float* bias, int renorm, int score, int groups, int keep, float w_scale, int has_gate, int32_t* ids,
+                               float* w, float* gate, int32_t* counts, void* stream) {
+  if (groups < 1 || keep < 1 || keep > groups || E_tot % groups || top > keep * (E_tot / groups))
+    return set_error(OMC_ERR_ARG, "omc_router_topk: equal groups, at least `top` outputs in the kept ones");
   if (score != OMC_ROUTER_SOFTMAX && score != OMC_ROUTER_SIGMOID) return set_error(OMC_ERR_ARG, "omc_router_topk: unknown score function");
   if (z == nullptr || ids == nullptr || w == nullptr || counts == nullptr || T < 0 || E_tot <= 0 || experts < 0 || experts > E_tot ||
       top <= 0 || top > E_tot || (has_gate && gate == nullptr))
     return set_error(OMC_ERR_ARG, "omc_router_topk: bad argument");
   if (E_tot > 4096 || top > 32) return set_error(OMC_ERR_SHAPE, "omc_router_topk: more than 4096 router outputs or top above 32");
   if (T == 0) return OMC_OK;
-  const size_t smem = sizeof(float) * 2 * (size_t)E_tot * kRouteWarps;
+  const size_t smem = sizeof(float) * (2 * (size_t)E_tot + groups) * kRouteWarps;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(router_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return set_error(OMC_ERR_CUDA, cudaGetErrorString(e));
   }
   router_topk_kernel<<<(T + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, static_cast<cudaStream_t>(stream)>>>(
-      z, ldz, T, E_tot, experts, top, correction, bias, renorm, score, has_gate, ids, w, gate, counts);
+      z, ldz, T, E_tot, experts, top, correction, bias, renorm, score, groups, keep, w_scale, has_gate, ids, w, gate, counts);
   return check_launch("omc_router_topk");
 }
 

@@ -211,6 +211,164 @@ __global__ void __launch_bounds__(256) tanh_cap_rows_kernel(float* __restrict__ 
   *p = cap * tanhf(*p / cap);
 }
 
+// ---- layer norm after the residual sum --------------------------------------------------------------------------------------
+//   v = alpha * x[t] + y[t] + sum_j w[t, j] * ys[slot_of[t, j]]        (y, ys: absent terms are zero)
+//   o = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * nw + nb    -> x_out[t] (fp32 stream), xb[t] (rounded: the next input)
+// One CTA per row; a thread keeps its NV float4 pieces of the row in registers (the variance is taken about the mean, two block
+// reductions with one barrier each). Rows that are not laid out for float4 or too wide go through shared memory instead (VEC false).
+struct LnResArgs {
+  const float* x;
+  long long ldx;
+  float alpha;
+  const float* y;
+  long long ldy;
+  const float* ys;
+  long long ldys;
+  const int32_t* slot_of;
+  const float* w;
+  int top;
+  const void* nw;
+  const void* nb;
+  float eps;
+  float* x_out;
+  long long ldxo;
+  void* xb;
+  long long ldxb;
+  int C;
+};
+
+template <int NT>
+__device__ __forceinline__ float row_sum(float v, float* red) {  // red: a [NT / 32] piece of shared memory no other reduction uses
+  v = seq_warp_sum(v);
+  if (NT == 32) return v;
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NT / 32; ++i) s += red[i];
+  return s;
+}
+
+template <typename TW, typename TB, int NT, int NV>
+__global__ void __launch_bounds__(NT) ln_residual_kernel(LnResArgs a) {
+  __shared__ float red[2][NT / 32];
+  const long long t = blockIdx.x;
+  float4 v[NV];
+  const float* xr = a.x + t * a.ldx;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * NT + threadIdx.x) * 4;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < a.C) {
+      const float4 q = *reinterpret_cast<const float4*>(xr + c);
+      v[i] = make_float4(a.alpha * q.x, a.alpha * q.y, a.alpha * q.z, a.alpha * q.w);
+      if (a.y != nullptr) {
+        const float4 u = *reinterpret_cast<const float4*>(a.y + t * a.ldy + c);
+        v[i].x += u.x, v[i].y += u.y, v[i].z += u.z, v[i].w += u.w;
+      }
+    }
+  }
+  if (a.ys != nullptr) {
+#pragma unroll 4
+    for (int k = 0; k < a.top; ++k) {
+      const int sl = a.slot_of[t * a.top + k];
+      if (sl < 0) continue;
+      const float wk = a.w[t * a.top + k];
+      const float* yr = a.ys + (long long)sl * a.ldys;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * NT + threadIdx.x) * 4;
+        if (c < a.C) {
+          const float4 u = *reinterpret_cast<const float4*>(yr + c);
+          v[i].x = fmaf(wk, u.x, v[i].x), v[i].y = fmaf(wk, u.y, v[i].y), v[i].z = fmaf(wk, u.z, v[i].z), v[i].w = fmaf(wk, u.w, v[i].w);
+        }
+      }
+    }
+  }
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+  const float mean = row_sum<NT>(s, red[0]) / (float)a.C;
+  s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    if ((i * NT + (int)threadIdx.x) * 4 < a.C) {
+      v[i].x -= mean, v[i].y -= mean, v[i].z -= mean, v[i].w -= mean;
+      s = fmaf(v[i].x, v[i].x, s), s = fmaf(v[i].y, v[i].y, s), s = fmaf(v[i].z, v[i].z, s), s = fmaf(v[i].w, v[i].w, s);
+    }
+  }
+  const float rstd = 1.f / sqrtf(row_sum<NT>(s, red[1]) / (float)a.C + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * NT + threadIdx.x) * 4;
+    if (c < a.C) {
+      float w4[4], b4[4];
+      ld4(static_cast<const TW*>(a.nw) + c, w4);
+      ld4(static_cast<const TW*>(a.nb) + c, b4);
+      const float o[4] = {fmaf(v[i].x * rstd, w4[0], b4[0]), fmaf(v[i].y * rstd, w4[1], b4[1]), fmaf(v[i].z * rstd, w4[2], b4[2]),
+                          fmaf(v[i].w * rstd, w4[3], b4[3])};
+      if (a.x_out != nullptr) st4(a.x_out + t * a.ldxo + c, o);
+      if (a.xb != nullptr) st4(static_cast<TB*>(a.xb) + t * a.ldxb + c, o);
+    }
+  }
+}
+
+template <typename TW, typename TB>
+__global__ void __launch_bounds__(256) ln_residual_any_kernel(LnResArgs a) {
+  extern __shared__ float row[];  // [C]
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  float s = 0.f;
+  for (int c = threadIdx.x; c < a.C; c += blockDim.x) {
+    float v = a.alpha * a.x[t * a.ldx + c];
+    if (a.y != nullptr) v += a.y[t * a.ldy + c];
+    if (a.ys != nullptr)
+      for (int k = 0; k < a.top; ++k) {
+        const int sl = a.slot_of[t * a.top + k];
+        if (sl >= 0) v = fmaf(a.w[t * a.top + k], a.ys[(long long)sl * a.ldys + c], v);
+      }
+    row[c] = v;
+    s += v;
+  }
+  const float mean = block_sum(s, red) / (float)a.C;
+  s = 0.f;
+  for (int c = threadIdx.x; c < a.C; c += blockDim.x) {   // every thread rereads only what it wrote
+    const float d = row[c] - mean;
+    s = fmaf(d, d, s);
+  }
+  const float rstd = 1.f / sqrtf(block_sum(s, red) / (float)a.C + a.eps);
+  for (int c = threadIdx.x; c < a.C; c += blockDim.x) {
+    const float o = fmaf((row[c] - mean) * rstd, ldf(static_cast<const TW*>(a.nw) + c), ldf(static_cast<const TW*>(a.nb) + c));
+    if (a.x_out != nullptr) a.x_out[t * a.ldxo + c] = o;
+    if (a.xb != nullptr) stf(static_cast<TB*>(a.xb) + t * a.ldxb + c, o);
+  }
+}
+
+template <typename TW, typename TB>
+static int launch_ln_residual(const LnResArgs& a, int rows, cudaStream_t st) {
+  auto al = [](const void* p, size_t n) { return p == nullptr || reinterpret_cast<uintptr_t>(p) % n == 0; };
+  const bool vec = a.C % 4 == 0 && a.C <= 8192 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ldys % 4 == 0 && a.ldxo % 4 == 0 && a.ldxb % 4 == 0 &&
+                   al(a.x, 16) && al(a.y, 16) && al(a.ys, 16) && al(a.x_out, 16) && al(a.nw, 4 * sizeof(TW)) && al(a.nb, 4 * sizeof(TW)) &&
+                   al(a.xb, 4 * sizeof(TB));
+  if (vec) {
+    if (a.C <= 256) ln_residual_kernel<TW, TB, 64, 1><<<rows, 64, 0, st>>>(a);
+    else if (a.C <= 512) ln_residual_kernel<TW, TB, 128, 1><<<rows, 128, 0, st>>>(a);
+    else if (a.C <= 1024) ln_residual_kernel<TW, TB, 256, 1><<<rows, 256, 0, st>>>(a);
+    else if (a.C <= 2048) ln_residual_kernel<TW, TB, 256, 2><<<rows, 256, 0, st>>>(a);
+    else if (a.C <= 4096) ln_residual_kernel<TW, TB, 256, 4><<<rows, 256, 0, st>>>(a);
+    else ln_residual_kernel<TW, TB, 256, 8><<<rows, 256, 0, st>>>(a);
+  } else {
+    const size_t smem = (size_t)a.C * sizeof(float);
+    if (smem > 200 * 1024) return set_error(OMC_ERR_SHAPE, "omc_ln_residual: row too wide for shared memory");
+    if (smem > 48 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(ln_residual_any_kernel<TW, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return set_error(OMC_ERR_CUDA, cudaGetErrorString(e));
+    }
+    ln_residual_any_kernel<TW, TB><<<rows, 256, smem, st>>>(a);
+  }
+  return check_launch("omc_ln_residual");
+}
+
 }  // namespace omc
 
 using namespace omc;
@@ -314,4 +472,17 @@ extern "C" int omc_tanh_cap_rows(float* x, long long ldx, int rows, int cols, fl
   const long long total = (long long)rows * cols;
   tanh_cap_rows_kernel<<<(unsigned)((total + 255) / 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(x, ldx, cols, total, cap);
   return check_launch("omc_tanh_cap_rows");
+}
+
+extern "C" int omc_ln_residual(const float* x, long long ldx, float alpha, const float* y, long long ldy, const float* ys, long long ldys,
+                               const int32_t* slot_of, const float* w, int top, const void* nw, const void* nb, int w_dt, float eps,
+                               float* x_out, long long ldxo, void* xb, int xb_dt, long long ldxb, int rows, int C, void* stream) {
+  if (x == nullptr || nw == nullptr || nb == nullptr || (x_out == nullptr && xb == nullptr) || rows < 0 || C <= 0 ||
+      (ys != nullptr && (slot_of == nullptr || w == nullptr || top <= 0)))
+    return set_error(OMC_ERR_ARG, "omc_ln_residual: bad argument");
+  if (rows == 0) return OMC_OK;
+  const LnResArgs a{x, ldx, alpha, y, y != nullptr ? ldy : 0, ys, ys != nullptr ? ldys : 0, slot_of, w, top, nw, nb, eps, x_out,
+                    x_out != nullptr ? ldxo : 0, xb, xb != nullptr ? ldxb : 0, C};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(xb_dt, TB, { return (launch_ln_residual<TW, TB>(a, rows, st)); }))
 }

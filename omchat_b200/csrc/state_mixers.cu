@@ -14,6 +14,7 @@
 // both columns, and a key or query value read from shared memory is used twice), and the eight lanes of a column pair finish the
 // two dot products of a token with three shuffles each. Tokens are staged 16 at a time in shared memory by cp.async, one chunk ahead of the one being
 // computed (decays, sigmoid and silu applied in place on arrival), so the sequential loop touches registers and shared memory only.
+// Recurrences whose channels carry one or a few states of their own (selective scan, gated linear recurrent unit) follow below.
 #include "seq_common.cuh"
 
 namespace omc {
@@ -704,6 +705,111 @@ __global__ void __launch_bounds__(kSelThreads) selective_scan_kernel(SelArgs a) 
   }
 }
 
+// ---- real-gated linear recurrent unit -------------------------------------------------------------------------------------
+// Per channel one state:  S <- a S + sqrt(1 - a^2) i u,  log a = -k r softplus(lam),  r and i sigmoids of raw gates that a block-
+// diagonal product left in g. Nothing couples the channels, and the recurrence is linear in S: a CTA owns blockDim.x channels of one
+// portion and blockDim.y consecutive runs of K tokens. Every thread evaluates its K tokens' (expm1(log a), input) in registers, runs
+// them from a zero state, and leaves (sum of log a, local state) of its run in shared memory; with the runs in front of its own it
+// gets its start state and goes over its K tokens once more from registers. A run's whole decay is applied as expm1 of the summed
+// log a - never as a product of rounded decays - so the state keeps its digits however the tokens are spread over threads. The output
+// is multiplied by gelu of the other branch. FAST (bf16 operands): hardware exponential, reciprocal and square root.
+constexpr int kLruTok = 8;
+
+struct LruArgs {
+  const void* u;
+  long long ldu;
+  const float* g;
+  long long ldg;
+  const float* gb;
+  const float* lam;
+  const float* y;
+  long long ldy;
+  float* state;
+  void* out;
+  long long ldo;
+  const int32_t* row_begin;
+  const int32_t* pos;
+  const int32_t* slot;
+  int width, n;   // n: channels per gate block
+  float scale;
+};
+
+template <bool FAST>
+__device__ __forceinline__ float lru_sigmoid(float z) { return FAST ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z); }
+template <bool FAST>
+__device__ __forceinline__ float lru_sqrt(float z) {
+  if (!FAST) return sqrtf(z);
+  float r;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(z));
+  return r;
+}
+template <bool FAST>
+__device__ __forceinline__ float lru_gelu(float z) {
+  const float p = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return 0.5f * z * (1.f + (FAST ? 1.f - __fdividef(2.f, __expf(2.f * p) + 1.f) : tanhf(p)));
+}
+template <bool FAST>
+__device__ __forceinline__ float lru_expm1(float x) { return FAST ? expm1_decay_f(x) : expm1f(x); }
+
+template <typename TD, bool FAST, int K>
+__global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
+  extern __shared__ float2 s_run[];  // [2][blockDim.y][blockDim.x]: (expm1 of the run's summed log a, its state from zero)
+  const int cx = threadIdx.x, wy = threadIdx.y, CX = blockDim.x, W = blockDim.y;
+  const int c = blockIdx.x * CX + cx;
+  const bool live = c < a.width;
+  const int r0 = a.row_begin[blockIdx.y], r1 = a.row_begin[blockIdx.y + 1];
+  if (r1 <= r0) return;
+  const bool fresh = a.pos[r0] == 0;
+  float* Sp = a.state + (long long)a.slot[r0] * a.width + c;
+  float carry = (live && !fresh) ? *Sp : 0.f;
+  const int blk = live ? c / a.n : 0, gr = blk * 2 * a.n + (live ? c - blk * a.n : 0), gi = gr + a.n;
+  const float sp = live ? -a.scale * softplus_f(a.lam[c]) : 0.f;
+  const float br = (live && a.gb != nullptr) ? a.gb[gr] : 0.f, bi = (live && a.gb != nullptr) ? a.gb[gi] : 0.f;
+  const TD* ug = static_cast<const TD*>(a.u);
+  TD* og = static_cast<TD*>(a.out);
+  int buf = 0;
+  for (int t0 = r0; t0 < r1; t0 += W * K, buf ^= 1) {
+    const int tb = t0 + wy * K;
+    float am1[K], in[K], yv[K];
+    float L = 0.f, loc = 0.f;
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+      am1[k] = in[k] = yv[k] = 0.f;
+      const long long t = tb + k;
+      if (live && t < r1) {
+        const float zr = a.g[t * a.ldg + gr], zi = a.g[t * a.ldg + gi], uv = ldf(ug + t * a.ldu + c);
+        if (a.y != nullptr) yv[k] = a.y[t * a.ldy + c];
+        const float la = sp * lru_sigmoid<FAST>(zr + br);
+        am1[k] = lru_expm1<FAST>(la);
+        in[k] = lru_sqrt<FAST>(-am1[k] * (2.f + am1[k])) * (lru_sigmoid<FAST>(zi + bi) * uv);
+        L += la;
+        loc = fmaf(am1[k], loc, loc) + in[k];
+      }
+    }
+    float S = carry;
+    if (W > 1) {
+      float2* run = s_run + (size_t)buf * W * CX;
+      run[wy * CX + cx] = make_float2(lru_expm1<FAST>(L), loc);
+      __syncthreads();   // the other buffer is rewritten only behind the next tile's barrier, which every reader of this one reaches first
+      for (int w = 0; w < W; ++w) {
+        if (w == wy) S = carry;
+        const float2 v = run[w * CX + cx];
+        carry = fmaf(v.x, carry, carry) + v.y;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+      const long long t = tb + k;
+      if (live && t < r1) {
+        S = fmaf(am1[k], S, S) + in[k];
+        stf(og + t * a.ldo + c, a.y != nullptr ? S * lru_gelu<FAST>(yv[k]) : S);
+      }
+    }
+    if (W == 1) carry = S;
+  }
+  if (live && wy == 0) *Sp = carry;
+}
+
 }  // namespace omc
 
 using namespace omc;
@@ -910,4 +1016,32 @@ extern "C" int omc_selective_scan(const void* x, int x_dt, long long ldx, const 
   }
 #undef OMC_SEL_LAUNCH
   return check_launch("omc_selective_scan");
+}
+
+template <typename TD, bool FAST>
+static int launch_rglru(const LruArgs& a, int rows, int portions, cudaStream_t st) {
+  // how many runs of tokens a CTA works on at once, by the average length of a portion (any choice is right for any length)
+  const int avg = (rows + portions - 1) / portions;
+  if (avg <= 2) {
+    rglru_scan_kernel<TD, FAST, 1><<<dim3((a.width + 127) / 128, portions), dim3(128, 1), 0, st>>>(a);
+  } else {
+    const int W = avg >= 96 ? 16 : (avg >= 24 ? 4 : 2);
+    rglru_scan_kernel<TD, FAST, kLruTok><<<dim3((a.width + 31) / 32, portions), dim3(32, W), (size_t)2 * W * 32 * sizeof(float2), st>>>(a);
+  }
+  return check_launch("omc_rglru_scan");
+}
+
+extern "C" int omc_rglru_scan(const void* u, int dt, long long ldu, const float* g, long long ldg, const float* gb, const float* lam,
+                              const float* y, long long ldy, float* state, void* out, long long ldo, const int32_t* row_begin, int portions,
+                              const int32_t* pos, const int32_t* slot, int rows, int width, int blocks, float decay_scale, void* stream) {
+  if (u == nullptr || g == nullptr || lam == nullptr || state == nullptr || out == nullptr || row_begin == nullptr || pos == nullptr ||
+      slot == nullptr || portions < 0 || rows < portions || width <= 0 || blocks <= 0 || width % blocks)
+    return set_error(OMC_ERR_ARG, "omc_rglru_scan: bad argument");
+  if (portions == 0) return OMC_OK;
+  if (portions > 65535) return set_error(OMC_ERR_SHAPE, "omc_rglru_scan: more than 65535 portions");
+  const LruArgs a{u, ldu, g, ldg, gb, lam, y, ldy, state, out, ldo, row_begin, pos, slot, width, width / blocks, decay_scale};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dt == OMC_DT_F32) return launch_rglru<float, false>(a, rows, portions, st);
+  if (dt == OMC_DT_BF16) return launch_rglru<bf16_t, true>(a, rows, portions, st);
+  return set_error(OMC_ERR_ARG, "omc_rglru_scan: unknown dtype code");
 }

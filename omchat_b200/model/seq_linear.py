@@ -1,4 +1,4 @@
-"""The linear layer of the sequence-step decoders (Voduzen, Tifisun, Fofisun): which kernel multiplies which matrix.
+"""The linear layer of the sequence-step decoders (Voduzen, Tifisun, Fofisun, Vefunex, Munevik): which kernel multiplies which matrix.
 
 Matrices with at least TENSOR_GEMM_MIN_WEIGHT elements go through the tcgen05 GEMM of the core library when the operands are bf16
 and the dimensions are multiples of 8; below it a launch is latency-bound either way and the kernel of the sequence-step library
@@ -10,7 +10,7 @@ that does not depend on M.
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Sequence
 
 import torch
 
@@ -35,3 +35,15 @@ def dense_linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, *, te
         return y if alpha == 1.0 else y.mul_(alpha)
     out = torch.empty(M, N, device=x.device, dtype=out_dtype)
     return seqlib.linear(x, w, out, alpha=alpha, act=act, bias=bias)
+
+
+def stack_rows(parts: Sequence[tuple]):
+    """[(name, matrix [n_i, C])] -> (stacked matrix with zero rows up to a multiple of 8, {name: column slice of its output})."""
+    cols, rows, at = {}, [], 0
+    for name, m in parts:
+        cols[name] = slice(at, at + m.shape[0])
+        at += m.shape[0]
+        rows.append(m)
+    if at % 8:   # the tensor-core GEMMs take N % 8 == 0; the extra outputs are never read
+        rows.append(torch.zeros(8 - at % 8, rows[0].shape[1], device=rows[0].device, dtype=rows[0].dtype))
+    return torch.cat(rows, dim=0).contiguous(), cols

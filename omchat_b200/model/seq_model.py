@@ -37,22 +37,27 @@ def portion_starts(decoder, T: int, slot: torch.Tensor, portions: Optional[Seque
 
 class GraphedDecodeMixin:
     """decode_step(): a step of one row per request, captured once per (rows, cache) and replayed. Every kernel of such a step
-    takes positions and slots from device memory and no launch shape depends on the contexts' lengths, so one capture serves
-    while the requests grow."""
+    takes positions and slots from device memory, so one capture serves while the requests grow; what launch shapes depend on the
+    contexts' lengths nevertheless a decoder names in decode_shape(), as a few coarse keyword arguments of its step()."""
 
     class _Graph:
         pass
 
     def _init_graphs(self):
-        self._graphs = {}         # (rows, id(cache)) -> captured decode-only step
+        self._graphs = {}         # (rows, id(cache), decode_shape) -> captured decode-only step
         self.use_graph = True
+
+    def decode_shape(self, B: int, max_keys: int) -> dict:
+        """Keyword arguments of step() that the launch shapes of a decode-only step of B rows over up to max_keys tokens depend on."""
+        return {}
 
     @torch.no_grad()
     def decode_step(self, meta_host: torch.Tensor, cache, max_keys: int) -> torch.Tensor:
         """meta_host int32 [3, B] (tokens, positions, slots; pinned host memory), one row per request. Returns fp32 logits
         [B, vocab] (a static buffer, overwritten by the next call)."""
         B = meta_host.shape[1]
-        key = (B, id(cache))
+        shape = self.decode_shape(B, max_keys)
+        key = (B, id(cache), tuple(sorted(shape.items())))
         g = self._graphs.get(key)
         if g is not None and g.cache is not cache:
             g = None
@@ -72,18 +77,18 @@ class GraphedDecodeMixin:
                 scratch = self.new_cache(2, cache.n_slots, 1)
                 dummy = torch.zeros(3, B, device=self.device, dtype=torch.int32)
                 dummy[2] = torch.arange(B, device=self.device, dtype=torch.int32) % cache.n_slots
-                self.step(dummy[0], dummy[1], dummy[2], scratch, g.want, one_row_each=True)
+                self.step(dummy[0], dummy[1], dummy[2], scratch, g.want, one_row_each=True, **shape)
                 torch.cuda.synchronize()
                 del scratch, dummy
                 n0 = lib.launch_count()
                 g.graph = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(g.graph):
-                    g.logits = self.step(g.meta[0], g.meta[1], g.meta[2], cache, g.want, one_row_each=True)
+                    g.logits = self.step(g.meta[0], g.meta[1], g.meta[2], cache, g.want, one_row_each=True, **shape)
                 g.launches = lib.launch_count() - n0
                 lib.add_launches(-g.launches)   # the capture does not execute
         g.meta.copy_(meta_host, non_blocking=True)
         if g.graph is None:
-            return self.step(g.meta[0], g.meta[1], g.meta[2], cache, g.want, one_row_each=True)
+            return self.step(g.meta[0], g.meta[1], g.meta[2], cache, g.want, one_row_each=True, **shape)
         g.graph.replay()
         lib.add_launches(g.launches)
         return g.logits

@@ -32,7 +32,7 @@ import torch
 from .. import seqlib
 from ..config import AttentionScanMixerSpec, GatedLinearAttentionSpec, SigmoidMoeSpec, SoftmaxAttentionSpec, VefunexConfig
 from .paged_cache import PagedStateCache
-from .seq_linear import dense_linear
+from .seq_linear import dense_linear, stack_rows
 from .seq_model import GraphedDecodeMixin, SequenceStepLM, portion_starts
 from .seq_moe import expert_workspace, grouped_tensor_gemm_ok, run_sorted_experts
 
@@ -109,18 +109,6 @@ class VefunexW:
     layers: List[VefunexLayerW]
 
 
-def _stack(parts: Sequence[tuple], device, dtype):
-    """[(name, matrix [n_i, C])] -> (stacked matrix with zero rows up to a multiple of 8, {name: column slice of its output})."""
-    cols, rows, at = {}, [], 0
-    for name, m in parts:
-        cols[name] = slice(at, at + m.shape[0])
-        at += m.shape[0]
-        rows.append(m)
-    if at % 8:   # the tensor-core GEMMs take N % 8 == 0; the extra outputs are never read
-        rows.append(torch.zeros(8 - at % 8, rows[0].shape[1], device=device, dtype=dtype))
-    return torch.cat(rows, dim=0).contiguous(), cols
-
-
 def weights_from_state_dict(sd: Dict[str, torch.Tensor], cfg: VefunexConfig, device, dtype: torch.dtype) -> VefunexW:
     """Checkpoint names: 'embed', 'final.norm' (+ '.b', '.alpha'), per layer i 'l<i>.norm1|norm2' (+ '.b', '.alpha'), 'l<i>.canon1|canon2',
     'l<i>.dwa', 'l<i>.mix.*', 'l<i>.mlp.router', 'l<i>.mlp.e<j>.gate|up|down'; linear weights [out, in]. Load-time re-layouts: one
@@ -149,7 +137,7 @@ def weights_from_state_dict(sd: Dict[str, torch.Tensor], cfg: VefunexConfig, dev
         parts = [("q", gs(p + "q", (nq, C))), ("k", gs(p + "k", (nk, C))), ("v", gs(p + "v", (nv, C)))]
         if a.gate:
             parts.append(("g", gs(p + "g", (a.heads * a.vdim, C))))
-        w_in, cols = _stack(parts + list(extra), device, dtype)
+        w_in, cols = stack_rows(parts + list(extra))
         return AttentionW(w_in=w_in, cols=cols, o=gs(p + "o", (C, a.heads * a.vdim)),
                           freq=seqlib.rotary_frequencies(a.rot.dims, a.rot.base, device) if a.rot is not None and a.rot.dims else None,
                           sink=gs(p + "sink", (a.heads,), f32) if a.sink else None)
@@ -163,8 +151,8 @@ def weights_from_state_dict(sd: Dict[str, torch.Tensor], cfg: VefunexConfig, dev
         elif isinstance(m, AttentionScanMixerSpec):
             r, q = m.right, p + "right."
             wx = gs(q + "x", (r.dt_rank + 2 * r.state, r.inner))
-            x_dt, _ = _stack([("dt", wx[:r.dt_rank])], device, dtype)
-            x_bc, _ = _stack([("bc", wx[r.dt_rank:])], device, dtype)
+            x_dt, _ = stack_rows([("dt", wx[:r.dt_rank])])
+            x_bc, _ = stack_rows([("bc", wx[r.dt_rank:])])
             right = ScanW(conv=gs(q + "conv", (r.inner, r.conv)), conv_b=gs(q + "conv.b", (r.inner,)), x_dt=x_dt, x_bc=x_bc,
                           dt=gs(q + "dt", (r.inner, r.dt_rank)),
                           dt_b=gs(q + "dt.b", (r.inner,), f32), A_log=gs(q + "A_log", (r.inner, r.state), f32), D=gs(q + "D", (r.inner,), f32),
@@ -174,15 +162,15 @@ def weights_from_state_dict(sd: Dict[str, torch.Tensor], cfg: VefunexConfig, dev
             assert isinstance(m, GatedLinearAttentionSpec)
             nqk, nv = m.heads * m.dim, m.heads * m.vdim
             a1 = g(p + "a1")
-            w_in, cols = _stack([("q", gs(p + "q", (nqk, C))), ("k", gs(p + "k", (nqk, C))), ("v", gs(p + "v", (nv, C))),
-                                 ("g", gs(p + "g", (nv, C)))], device, dtype)
-            a1s, _ = _stack([("a1", need(a1, (a1.shape[0], C), p + "a1"))], device, dtype)
+            w_in, cols = stack_rows([("q", gs(p + "q", (nqk, C))), ("k", gs(p + "k", (nqk, C))), ("v", gs(p + "v", (nv, C))),
+                                 ("g", gs(p + "g", (nv, C)))])
+            a1s, _ = stack_rows([("a1", need(a1, (a1.shape[0], C), p + "a1"))])
             mix = GlaW(w_in=w_in, cols=cols, a1=a1s, a2=gs(p + "a2", (nqk, a1.shape[0])), a2_b=gs(p + "a2.b", (nqk,), f32), norm=gs(p + "norm", (m.vdim,)),
                        o=gs(p + "o", (C, nv)))
         mlp, q = None, f"l{i}.mlp."
         if spec.mlp is not None:
             s = spec.mlp
-            router, _ = _stack([("r", gs(q + "router", (s.experts, C)))], device, dtype)
+            router, _ = stack_rows([("r", gs(q + "router", (s.experts, C)))])
             mlp = SigmoidMoeW(router=router,
                               gate_up=torch.stack([torch.cat([gs(f"{q}e{e}.gate", (s.expert_ff, C)), gs(f"{q}e{e}.up", (s.expert_ff, C))], dim=0)
                                                    for e in range(s.experts)]).contiguous(),

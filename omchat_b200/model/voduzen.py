@@ -25,8 +25,9 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from .. import lib, seqlib
-from ..config import LatentAttentionSpec, RouterMoeSpec, VoduzenConfig
+from ..config import RouterMoeSpec, VoduzenConfig
 from .paged_cache import PagedLatentCache
+from .seq_latent import LatentAttention
 from .seq_linear import TENSOR_GEMM_MIN_WEIGHT, dense_linear
 
 
@@ -44,7 +45,6 @@ class LatentAttnW:
     uv: torch.Tensor                # [H * dv, kv_rank]
     o: torch.Tensor                 # [C, H * dv]
     sink: Optional[torch.Tensor]    # fp32 [H]
-    rot_cs: torch.Tensor = None     # fp32 [positions, dims / 2, 2], grown on demand
 
 
 @dataclass
@@ -175,9 +175,8 @@ class VoduzenDecoder:
         self.C = cfg.hidden_size
         self.eps = cfg.norm_eps
         self.tensor_gemm = dtype == torch.bfloat16
-        self.tensor_attention = True    # False: the plain attention kernel for every shape (A/B, tests)
+        self.latent = LatentAttention(self.device, dtype)
         self._moe_ws = {}
-        self._decode_plans = {}   # (rows, heads, parts) -> seqlib.DecodeAttnPlan
         self._graphs = {}         # (rows, parts, id(cache)) -> captured decode-only step
         self.use_graph = True
 
@@ -189,18 +188,13 @@ class VoduzenDecoder:
         return PagedLatentCache(self.cache_widths(), n_pages, n_slots, self.cfg.kv_page_size, self.dtype, self.device,
                                 max_pages_per_slot)
 
-    def _rot_table(self, mw: LatentAttnW, spec: LatentAttentionSpec, positions: int) -> torch.Tensor:
-        """fp32 (cos, sin) [positions, dims / 2, 2]: angles and functions evaluated in double precision on the host, once."""
-        t = mw.rot_cs
-        if t is None or t.shape[0] < positions:
-            n = max(positions, 1024)
-            f, mult = spec.rot.frequencies()
-            ang = torch.arange(n, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)[None, :]
-            t = (torch.stack([ang.cos(), ang.sin()], dim=-1) * mult).to(torch.float32).contiguous().to(self.device)
-            if t.numel() == 0:   # no rotated dimensions: the kernels still want a valid pointer
-                t = torch.zeros(n, 1, 2, device=self.device)
-            mw.rot_cs = t
-        return t
+    @property
+    def tensor_attention(self) -> bool:
+        return self.latent.tensor_attention
+
+    @tensor_attention.setter
+    def tensor_attention(self, on: bool):
+        self.latent.tensor_attention = on
 
     # ---- linear layers
     def _linear(self, x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, act: int = seqlib.ACT_NONE, alpha: float = 1.0):
@@ -226,7 +220,7 @@ class VoduzenDecoder:
         else:
             q = self._linear(xb, mw.q, qdt)
             dkv32 = self._linear(xb, mw.dkv, f32)
-        cs = self._rot_table(mw, spec, cache.capacity)
+        cs = self.latent.rotary.get(spec.rot, cache.capacity)
         pool = cache.pools[li]
         qcat = torch.empty(T, H, r + dr, device=xb.device, dtype=self.dtype)
         # latent norm + key rotation + cache append + query rotation in one launch
@@ -235,22 +229,7 @@ class VoduzenDecoder:
         # absorbed keys: qcat[t, h, :r] = q[t, h, :dn] @ W_uk,h  (one problem per head, column slices of both buffers)
         seqlib.linear(q, mw.uk_t, qcat, M=T, N=r, K=dn, ldx=q.stride(0), sx=dn + dr, ldw=dn, sw=r * dn, ldy=H * (r + dr),
                       sy=r + dr, batch=H)
-        use_mma = plans is not None and self.tensor_attention and seqlib.latent_attn_mma_ok(H, r, dr, self.dtype)
-        olat = torch.empty(T, H, r, device=xb.device, dtype=self.dtype if use_mma else f32)
-        if use_mma:
-            plan = plans.get(H)
-            if plan is None:
-                if "decode_parts" in plans:       # decode-only step: the list is written on the device from pos / slot
-                    plan = self._decode_plans.get((T, H, plans["decode_parts"]))
-                    if plan is None:
-                        plan = self._decode_plans[(T, H, plans["decode_parts"])] = seqlib.DecodeAttnPlan(T, H, plans["decode_parts"], xb.device)
-                    plan.fill(pos, slot)
-                else:
-                    plan = seqlib.LatentAttnPlan(plans["portions"], H, xb.device)
-                plans[H] = plan
-            seqlib.latent_attn_mma(qcat, r, dr, pool, cache.block_table, cache.page_size, plan, mw.sink, spec.scale, olat)
-        else:
-            seqlib.latent_attn(qcat, r, dr, pool, cache.block_table, cache.page_size, pos, slot, mw.sink, spec.scale, olat)
+        olat = self.latent.attend(qcat, r, dr, pool, cache, pos, slot, plans, spec.scale, sink=mw.sink)
         # values: attn[t, h*dv:(h+1)*dv] = W_uv,h @ olat[t, h]
         attn = torch.empty(T, H * dv, device=xb.device, dtype=self.dtype)
         seqlib.linear(olat, mw.uv, attn, M=T, N=dv, K=r, ldx=H * r, sx=r, ldw=r, sw=dv * r, ldy=H * dv, sy=dv, batch=H)

@@ -47,17 +47,19 @@ SIGNATURES = {
     "omc_window_attn_mma": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _P, _I, _I, _F, _F, _P, _P, _P, _L, _I, _P, _I, _L, _P]),
     "omc_diff_attn_pair_ok": (_I, [_I, _I, _I, _I]),
     "omc_diff_attn_pair": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _I, _I, _F, _F, _F, _F, _P, _L, _I, _P, _I, _L, _P]),
+    "omc_ln_residual": (_I, [_P, _L, _F, _P, _L, _P, _L, _P, _P, _I, _P, _P, _I, _F, _P, _L, _P, _I, _L, _I, _I, _P]),
+    "omc_rglru_scan": (_I, [_P, _I, _L, _P, _L, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _F, _P]),
     "omc_embed_scale": (_I, [_P, _I, _P, _I, _I, _I, _F, _P, _L, _P, _I, _L, _P]),
     "omc_rms_rows": (_I, [_P, _L, _P, _I, _I, _F, _P, _I, _L, _I, _I, _P]),
     "omc_norm_residual": (_I, [_P, _L, _P, _I, _F, _P, _L, _P, _I, _L, _I, _I, _P]),
     "omc_latent_kv_store": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _I, _P, _P, _P, _I, _I, _P, _I, _P]),
-    "omc_latent_rope_store": (_I, [_P, _L, _I, _I, _I, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _I, _P, _I, _P]),
+    "omc_latent_rope_store": (_I, [_P, _L, _I, _I, _I, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _L, _I, _I, _P, _P, _I, _P]),
     "omc_moe_plan_scatter_small": (_I, [_P, _I, _I, _I, _P, _P, _P, _I, _L, _I, _I, _P, _I, _P, _P, _L, _P, _P]),
     "omc_rotary_q": (_I, [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P]),
-    "omc_latent_attn": (_I, [_P, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _P, _F, _P, _P]),
-    "omc_latent_attn_mma": (_I, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _I, _P, _F, _P, _I, _P, _P, _P]),
-    "omc_latent_decode_items": (_I, [_P, _P, _I, _I, _I, _P, _P, _P]),
-    "omc_router_topk": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P, _P, _P, _P, _P]),
+    "omc_latent_attn": (_I, [_P, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _P, _I, _P, _L, _F, _P, _P]),
+    "omc_latent_attn_mma": (_I, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _I, _P, _I, _P, _L, _F, _P, _I, _P, _P, _P]),
+    "omc_latent_decode_items": (_I, [_P, _P, _I, _I, _I, _I, _P, _P, _P]),
+    "omc_router_topk": (_I, [_P, _L, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P, _P]),
     "omc_moe_plan_tiles": (_I, [_P, _I, _I, _I, _P, _P, _P, _P]),
     "omc_moe_scatter_rows": (_I, [_P, _I, _L, _I, _I, _P, _I, _I, _P, _P, _P, _P, _L, _P, _P]),
     "omc_moe_combine_norm": (_I, [_P, _L, _P, _P, _I, _P, _P, _L, _P, _I, _F, _P, _L, _P, _P, _I, _L, _I, _I, _P]),
@@ -185,15 +187,18 @@ def latent_kv_store(dkv: torch.Tensor, r: int, dr: int, w: torch.Tensor, eps: fl
     _check(rc, "omc_latent_kv_store")
 
 
-def latent_rope_store(dkv, r: int, dr: int, w, eps: float, cs, rot_dims: int, pos, slot, block_table, page_size: int, pool, q, H: int,
-                      dn: int, qcat):
-    """latent_kv_store + rotary_q in one launch (w, pool, q, qcat of one dtype)."""
-    _need_cuda(dkv, w, cs, pos, slot, block_table, pool, q, qcat)
-    assert dkv.dtype == torch.float32 and w.dtype == pool.dtype == q.dtype == qcat.dtype and q.stride(1) == 1
-    assert block_table.is_contiguous() and pool.is_contiguous() and qcat.is_contiguous() and pool.shape[-1] == r + dr
-    rc = load().omc_latent_rope_store(_ptr(dkv), dkv.stride(0), dkv.shape[0], r, dr, _ptr(w), eps, _ptr(cs), rot_dims, _ptr(pos), _ptr(slot),
-                                      _ptr(block_table), block_table.shape[1], page_size, _ptr(pool), _ptr(q), q.stride(0), H, dn,
-                                      _ptr(qcat), _dt(pool), _stream())
+def latent_rope_store(dkv: Optional[torch.Tensor], r: int, dr: int, w, eps: float, cs, rot_dims: int, pos, slot, block_table, page_size: int, pool, q,
+                      H: int, dn: int, qcat, qn: Optional[torch.Tensor] = None):
+    """latent_kv_store + rotary_q in one launch (w, pool, qcat of one dtype, q of that dtype or fp32). dkv None: the queries only. qn
+    [T, H * dn]: receives the unrotated query parts."""
+    _need_cuda(dkv, w, cs, pos, slot, block_table, pool, q, qcat, qn)
+    assert qcat.is_contiguous() and q.stride(1) == 1 and (qn is None or (qn.is_contiguous() and qn.dtype == qcat.dtype and qn.shape[1] == H * dn))
+    if dkv is not None:
+        assert dkv.dtype == torch.float32 and dkv.stride(1) == 1 and w.dtype == pool.dtype == qcat.dtype
+        assert block_table.is_contiguous() and pool.is_contiguous() and pool.shape[-1] == r + dr
+    rc = load().omc_latent_rope_store(_ptr(dkv), dkv.stride(0) if dkv is not None else 0, q.shape[0], r, dr, _ptr(w), eps, _ptr(cs), rot_dims, _ptr(pos),
+                                      _ptr(slot), _ptr(block_table), block_table.shape[1], page_size, _ptr(pool), _ptr(q), _dt(q), q.stride(0), H, dn,
+                                      _ptr(qcat), _ptr(qn), _dt(qcat), _stream())
     _check(rc, "omc_latent_rope_store")
 
 
@@ -217,15 +222,22 @@ def rotary_q(q32: torch.Tensor, H: int, dn: int, dr: int, cs: torch.Tensor, rot_
     _check(rc, "omc_rotary_q")
 
 
+WINDOW_ALL = 1 << 30   # a window that never ends: plain causal attention
+
+
 def latent_attn(qcat: torch.Tensor, r: int, dr: int, pool: torch.Tensor, block_table: torch.Tensor, page_size: int,
-                pos: torch.Tensor, slot: torch.Tensor, sink: Optional[torch.Tensor], scale: float, out: torch.Tensor):
-    """qcat [T, H, r + dr] -> out fp32 [T, H, r] (weighted sums of cached latents)."""
-    _need_cuda(qcat, pool, block_table, pos, slot, sink, out)
+                pos: torch.Tensor, slot: torch.Tensor, sink: Optional[torch.Tensor], scale: float, out: torch.Tensor,
+                window: int = WINDOW_ALL, gate: Optional[torch.Tensor] = None):
+    """qcat [T, H, r + dr] -> out fp32 [T, H, r] (weighted sums of cached latents). window: keys a row sees behind itself, itself
+    included; gate fp32 [T, H]: head h's output is multiplied by sigmoid(gate[t, h])."""
+    _need_cuda(qcat, pool, block_table, pos, slot, sink, out, gate)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
     T, H = qcat.shape[0], qcat.shape[1]
     assert out.dtype == torch.float32 and out.is_contiguous() and qcat.is_contiguous()
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     rc = load().omc_latent_attn(_ptr(qcat), _dt(qcat), T, H, r, dr, _ptr(pool), _dt(pool), _ptr(block_table), block_table.shape[1],
-                                page_size, _ptr(pos), _ptr(slot), _ptr(sink), scale, _ptr(out), _stream())
+                                page_size, _ptr(pos), _ptr(slot), _ptr(sink), window, _ptr(gate), gate.stride(0) if gate is not None else 0, scale,
+                                _ptr(out), _stream())
     _check(rc, "omc_latent_attn")
     return out
 
@@ -248,7 +260,7 @@ class LatentAttnPlan:
 
     MAX_PARTS = 64  # key ranges one merge group may have (csrc/latent_attention.cu: kMergeMaxParts)
 
-    def __init__(self, portions, H: int, device, target_ctas: int = 296, min_keys: int = 128):
+    def __init__(self, portions, H: int, device, target_ctas: int = 296, min_keys: int = 128, window: int = WINDOW_ALL):
         import numpy as np
         tok = max(1, MMA_ROWS // H)
         base = sum(-(-n // tok) for _, n, _, _ in portions)
@@ -256,21 +268,23 @@ class LatentAttnPlan:
         for first_row, n, slot, p0 in portions:
             starts = np.arange(0, n, tok, dtype=np.int64)
             ntok = np.minimum(tok, n - starts)
-            keys = p0 + starts + ntok                                  # keys the tile's last row sees
+            ends = p0 + starts + ntok                                  # end of the keys the tile's last row sees
+            lows = np.maximum(0, p0 + starts - window + 1)             # first key its first row sees
+            keys = ends - lows
             parts = np.ones_like(starts)
             if base < target_ctas // 2:
                 parts = np.clip(np.minimum(-(-keys // min_keys), -(-target_ctas // max(base, 1))), 1, self.MAX_PARTS)
             for i in range(len(starts)):
-                np_i, k = int(parts[i]), int(keys[i])
+                np_i, k, lo = int(parts[i]), int(keys[i]), int(lows[i])
                 fr, nt = first_row + int(starts[i]), int(ntok[i])
                 if np_i == 1:
-                    items.append((fr, nt, slot, p0 + int(starts[i]), 0, k, -1, 0))
+                    items.append((fr, nt, slot, p0 + int(starts[i]), lo, lo + k, -1, 0))
                     continue
                 span = -(-(-(-k // np_i)) // MMA_ROWS) * MMA_ROWS       # keys per part, a multiple of 64
                 np_i = -(-k // span)
                 merges.append((fr * H, nt * H, part, np_i))
                 for j in range(np_i):
-                    items.append((fr, nt, slot, p0 + int(starts[i]), j * span, min(k, (j + 1) * span), part, 0))
+                    items.append((fr, nt, slot, p0 + int(starts[i]), lo + j * span, lo + min(k, (j + 1) * span), part, 0))
                     part += 1
         self.n_items, self.n_merges, self.n_parts = len(items), len(merges), part
         flat = torch.tensor(items, dtype=torch.int32).view(-1)
@@ -284,8 +298,8 @@ class DecodeAttnPlan:
     """Work list of a decode-only step of B rows with static device buffers: `fill(pos, slot)` rewrites it on the device each step
     (omc_latent_decode_items), so a captured CUDA graph stays valid while the contexts grow. parts: key ranges per row."""
 
-    def __init__(self, B: int, H: int, parts: int, device):
-        self.B, self.H, self.parts = B, H, parts
+    def __init__(self, B: int, H: int, parts: int, device, window: int = WINDOW_ALL):
+        self.B, self.H, self.parts, self.window = B, H, parts, window
         self.items = torch.zeros(B * parts * 8, device=device, dtype=torch.int32)
         self.merges = torch.zeros(B * 4, device=device, dtype=torch.int32) if parts > 1 else None
         self.n_items = B * parts
@@ -300,8 +314,8 @@ class DecodeAttnPlan:
         return max(1, min(bucket // min_keys, -(-target_ctas // B), LatentAttnPlan.MAX_PARTS))
 
     def fill(self, pos: torch.Tensor, slot: torch.Tensor):
-        rc = load().omc_latent_decode_items(_ptr(pos), _ptr(slot), self.B, self.H, self.parts, _ptr(self.items), _ptr(self.merges),
-                                            _stream())
+        rc = load().omc_latent_decode_items(_ptr(pos), _ptr(slot), self.B, self.H, self.parts, self.window, _ptr(self.items),
+                                            _ptr(self.merges), _stream())
         _check(rc, "omc_latent_decode_items")
 
 
@@ -309,8 +323,11 @@ _mma_ws = {}
 
 
 def latent_attn_mma(qcat: torch.Tensor, r: int, dr: int, pool: torch.Tensor, block_table: torch.Tensor, page_size: int,
-                    plan: LatentAttnPlan, sink: Optional[torch.Tensor], scale: float, out: torch.Tensor):
-    _need_cuda(qcat, pool, block_table, plan.items, sink, out)
+                    plan: LatentAttnPlan, sink: Optional[torch.Tensor], scale: float, out: torch.Tensor, window: int = WINDOW_ALL,
+                    gate: Optional[torch.Tensor] = None):
+    """latent_attn on the tensor cores; the plan was made for the same window."""
+    _need_cuda(qcat, pool, block_table, plan.items, sink, out, gate)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
     T, H = qcat.shape[0], qcat.shape[1]
     assert qcat.dtype == torch.bfloat16 and pool.dtype == torch.bfloat16
     assert qcat.is_contiguous() and out.is_contiguous() and pool.is_contiguous()
@@ -324,8 +341,8 @@ def latent_attn_mma(qcat: torch.Tensor, r: int, dr: int, pool: torch.Tensor, blo
             _mma_ws[key] = ws
         ws_o, ws_ml = ws[:plan.n_parts * MMA_ROWS * r], ws[plan.n_parts * MMA_ROWS * r:]
     rc = load().omc_latent_attn_mma(_ptr(qcat), T, H, r, dr, _ptr(pool), _ptr(block_table), block_table.shape[1], page_size,
-                                    _ptr(plan.items), plan.n_items, _ptr(plan.merges), plan.n_merges, _ptr(sink), scale, _ptr(out),
-                                    _dt(out), _ptr(ws_o), _ptr(ws_ml), _stream())
+                                    _ptr(plan.items), plan.n_items, _ptr(plan.merges), plan.n_merges, _ptr(sink), window, _ptr(gate),
+                                    gate.stride(0) if gate is not None else 0, scale, _ptr(out), _dt(out), _ptr(ws_o), _ptr(ws_ml), _stream())
     _check(rc, "omc_latent_attn_mma")
     if plan.n_merges:
         _core.add_launches(1)
@@ -334,15 +351,17 @@ def latent_attn_mma(qcat: torch.Tensor, r: int, dr: int, pool: torch.Tensor, blo
 
 def router_topk(z: torch.Tensor, e_tot: int, experts: int, top: int, correction: Optional[torch.Tensor], has_gate: bool,
                 ids: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor], counts: torch.Tensor,
-                bias: Optional[torch.Tensor] = None, renorm: bool = False, score: int = ROUTER_SOFTMAX):
+                bias: Optional[torch.Tensor] = None, renorm: bool = False, score: int = ROUTER_SOFTMAX, groups: int = 1, keep: int = 1,
+                scale: float = 1.0):
     """bias: fp32 [e_tot] added to the logits; renorm: the weights of the chosen are divided by their sum (softmax over the chosen);
-    score ROUTER_SIGMOID: every output is scored by a sigmoid of its own instead of the softmax over all."""
+    score ROUTER_SIGMOID: every output is scored by a sigmoid of its own instead of the softmax over all. groups / keep: only outputs
+    of the `keep` groups with the largest sums of their two best scores can be chosen; scale multiplies the weights."""
     _need_cuda(z, correction, bias, ids, w, gate, counts)
     assert z.dtype == torch.float32 and ids.dtype == torch.int32 and w.dtype == torch.float32 and counts.dtype == torch.int32
     assert correction is None or correction.dtype == torch.float32
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == e_tot)
     rc = load().omc_router_topk(_ptr(z), z.stride(0), z.shape[0], e_tot, experts, top, _ptr(correction), _ptr(bias), 1 if renorm else 0, score,
-                                1 if has_gate else 0, _ptr(ids), _ptr(w), _ptr(gate), _ptr(counts), _stream())
+                                groups, keep, scale, 1 if has_gate else 0, _ptr(ids), _ptr(w), _ptr(gate), _ptr(counts), _stream())
     _check(rc, "omc_router_topk")
 
 
@@ -410,6 +429,26 @@ def post_norm_residual(y1: torch.Tensor, w_post: torch.Tensor, eps: float, mult:
                                        _ptr(w_post), _dt(w_post), eps, mult, _ptr(h32), h32.stride(0), _ptr(w_next), _ptr(xb), _dt(xb),
                                        xb.stride(0) if xb is not None else 0, h32.shape[0], h32.shape[1], _stream())
     _check(rc, "omc_post_norm_residual")
+
+
+def ln_residual(x: torch.Tensor, alpha: float, nw: torch.Tensor, nb: torch.Tensor, eps: float, *, y: Optional[torch.Tensor] = None,
+                ys: Optional[torch.Tensor] = None, slot_of: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, top: int = 0,
+                x_out: Optional[torch.Tensor] = None, xb: Optional[torch.Tensor] = None):
+    """Layer norm of v = alpha x + y + sum_j w[t, j] ys[slot_of[t, j]] (absent terms are zero) with weight nw and bias nb -> x_out (fp32,
+    may be x) and / or xb (the rounded row)."""
+    _need_cuda(x, nw, nb, y, ys, slot_of, w, x_out, xb)
+    C = x.shape[1]
+    for t in (x, y, ys, x_out):
+        assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
+    assert nw.dtype == nb.dtype and nw.numel() == C and nb.numel() == C and (xb is None or xb.stride(1) == 1)
+    assert ys is None or (slot_of.is_contiguous() and w.is_contiguous() and w.dtype == torch.float32)
+
+    def ld(t):
+        return t.stride(0) if t is not None else 0
+    rc = load().omc_ln_residual(_ptr(x), ld(x), alpha, _ptr(y), ld(y), _ptr(ys), ld(ys), _ptr(slot_of), _ptr(w), top, _ptr(nw), _ptr(nb), _dt(nw), eps,
+                                _ptr(x_out), ld(x_out), _ptr(xb), _dt(xb), ld(xb), x.shape[0], C, _stream())
+    _check(rc, "omc_ln_residual")
+    return x_out if xb is None else xb
 
 
 def glu_mul(z: torch.Tensor, n: int, act: int, out: torch.Tensor, limit: float = 0.0, slope: float = 1.0, shift: float = 0.0):
@@ -528,9 +567,6 @@ def qk_norm_kv_store(q: torch.Tensor, wq: torch.Tensor, k: torch.Tensor, wk: tor
                                      nv, eps, q.shape[0], _ptr(pos), _ptr(slot), _ptr(block_table), block_table.shape[1], page_size,
                                      _ptr(pool), _ptr(q_out), q_out.stride(0), _dt(pool), _stream())
     _check(rc, "omc_qk_norm_kv_store")
-
-
-WINDOW_ALL = 1 << 30   # a window that never ends: plain causal attention
 
 
 def window_attn(q: torch.Tensor, H: int, G: int, d: int, dv: int, pool: torch.Tensor, block_table: torch.Tensor, page_size: int, pos, slot,
@@ -696,6 +732,25 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, B: 
                                    Cm.stride(0), _ptr(A_log), _ptr(D), _ptr(z), z.stride(0) if z is not None else 0, _ptr(state), _ptr(out),
                                    _dt(out), out.stride(0), _ptr(row_begin), portions, _ptr(pos), _ptr(slot), inner, N, _stream())
     _check(rc, "omc_selective_scan")
+    return out
+
+
+def rglru_scan(u: torch.Tensor, g: torch.Tensor, gb: Optional[torch.Tensor], lam: torch.Tensor, y: Optional[torch.Tensor], state: torch.Tensor,
+               out: torch.Tensor, row_begin: torch.Tensor, portions: int, pos, slot, blocks: int, decay_scale: float):
+    """The recurrence of omc_rglru_scan: u [T, width] (fp32 or bf16), raw gates g fp32 [T, 2 * width] with their biases gb, y fp32 rows
+    (a column slice is fine), state fp32 [slots, width] -> out [T, width] = S gelu(y)."""
+    _need_cuda(u, g, gb, lam, y, state, out, row_begin, pos, slot)
+    width = lam.numel()
+    assert u.dtype == out.dtype and u.stride(1) == 1 and out.stride(1) == 1 and u.shape[1] == width and g.shape[1] >= 2 * width
+    for t in (g, y):
+        assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
+    for t in (lam, gb):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (width,) and row_begin.dtype == torch.int32
+    rc = load().omc_rglru_scan(_ptr(u), _dt(u), u.stride(0), _ptr(g), g.stride(0), _ptr(gb), _ptr(lam), _ptr(y), y.stride(0) if y is not None else 0,
+                               _ptr(state), _ptr(out), out.stride(0), _ptr(row_begin), portions, _ptr(pos), _ptr(slot), u.shape[0], width, blocks,
+                               decay_scale, _stream())
+    _check(rc, "omc_rglru_scan")
     return out
 
 
