@@ -308,6 +308,10 @@ def main():
                     "this size (random weights; attention beside a selective scan, attention, gated linear attention, experts) beside "
                     "the Tifisun decoder at equal size - prefill and decode throughput and the new kernels against their rooflines "
                     "(tools/bench_vefunex.py); one JSON line per size")
+    ap.add_argument("--munevik", action="append", choices=["s", "m"], help="instead of the default workload: the Munevik decoder at "
+                    "this size (random weights; gated linear recurrent layers, windowed latent attention, dense and group-limited expert "
+                    "feed-forwards) beside the Voduzen decoder at equal size - prefill and decode throughput and the new kernels against "
+                    "their rooflines (tools/bench_munevik.py); one JSON line per size")
     ap.add_argument("--pixel-shuffle", type=float, default=1.0, help="mm_pixel_shuffle_ratio (1.0 = reference behaviour)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -343,6 +347,14 @@ def main():
         torch.cuda.set_device(0)
         for size in args.vefunex:
             print(json.dumps(measure_vefunex(size, steps=max(args.steps, 8))), flush=True)
+        return
+
+    if args.munevik:
+        import torch
+        from tools.bench_munevik import measure as measure_munevik
+        torch.cuda.set_device(0)
+        for size in args.munevik:
+            print(json.dumps(measure_munevik(size, steps=max(args.steps, 8))), flush=True)
         return
 
     import torch

@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
   const int p = pos[t];
   const int half = rot_dims >> 1;
   const float* csr = cs + (long long)p * rot_dims;
-  if (dkv != nullptr) {
+  if (dkv != nullptr && blockIdx.y == 0) {
     const float* row = dkv + (long long)t * ld;
     const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
     T* dst = pool + ((long long)page * page_size + p % page_size) * (r + dr);
@@ -96,9 +96,10 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
     }
     for (int c = rot_dims + threadIdx.x; c < dr; c += blockDim.x) stf(dst + r + c, row[r + c]);
   }
-  // queries: every (head, pair) is one unit of work
-  for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
-    const int h = i / half, j = i - h * half;
+  // queries: every (head, pair) is one unit of work; on short steps the heads are spread over blockIdx.y
+  const int per = (H + gridDim.y - 1) / gridDim.y, h0 = blockIdx.y * per, nh = min(per, H - h0);
+  for (int i = threadIdx.x; i < nh * half; i += blockDim.x) {
+    const int h = h0 + i / half, j = i % half;
     const TQ* src = q + (long long)t * ldq + (long long)h * (dn + dr) + dn;
     T* qd = qcat + ((long long)t * H + h) * (r + dr) + r;
     const float u = ldf(src + 2 * j), v = ldf(src + 2 * j + 1), co = csr[2 * j], si = csr[2 * j + 1];
@@ -106,14 +107,14 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
     stf(qd + 2 * j + 1, v * co + u * si);
   }
   const int rest = dr - rot_dims;
-  for (int i = threadIdx.x; i < H * rest; i += blockDim.x) {
-    const int h = i / rest, c = rot_dims + (i - h * rest);
+  for (int i = threadIdx.x; i < nh * rest; i += blockDim.x) {
+    const int h = h0 + i / rest, c = rot_dims + i % rest;
     stf(qcat + ((long long)t * H + h) * (r + dr) + r + c, ldf(q + (long long)t * ldq + (long long)h * (dn + dr) + dn + c));
   }
   if (qn != nullptr) {
-    for (int i = threadIdx.x; i < H * dn; i += blockDim.x) {
-      const int h = i / dn, c = i - h * dn;
-      stf(qn + (long long)t * H * dn + i, ldf(q + (long long)t * ldq + (long long)h * (dn + dr) + c));
+    for (int i = threadIdx.x; i < nh * dn; i += blockDim.x) {
+      const int h = h0 + i / dn, c = i % dn;
+      stf(qn + ((long long)t * H + h) * dn + c, ldf(q + (long long)t * ldq + (long long)h * (dn + dr) + c));
     }
   }
 }
@@ -230,7 +231,7 @@ extern "C" int omc_latent_rope_store(const float* dkv, long long ld, int T, int 
   if (T == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   OMC_DT_SWITCH(dt, TT, OMC_DT_SWITCH(q_dt, TQ, {
-    latent_rope_store_kernel<TT, TQ><<<T, 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, pos, slot, block_table,
+    latent_rope_store_kernel<TT, TQ><<<dim3(T, T <= 64 ? (H + 3) / 4 : 1), 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, pos, slot, block_table,
                                                         max_pages, page_size, static_cast<TT*>(pool), static_cast<const TQ*>(q), ldq, H, dn,
                                                         static_cast<TT*>(qcat), static_cast<TT*>(qn));
   }))

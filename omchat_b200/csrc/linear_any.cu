@@ -94,16 +94,6 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(LinearArgs a) {
 // steps of a few rows, where there are few row blocks to fill the device with).
 constexpr int kNarrowRows = 8, kNarrowMaxN = 64, kNarrowKC = 1024, kNarrowPerWarp = kNarrowMaxN / 8;
 
-__device__ __forceinline__ void nld4(const float* p, float (&v)[4]) {
-  const float4 t = *reinterpret_cast<const float4*>(p);
-  v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
-}
-__device__ __forceinline__ void nld4(const bf16_t* p, float (&v)[4]) {
-  const uint2 t = *reinterpret_cast<const uint2*>(p);
-  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
-  v[0] = lo.x, v[1] = lo.y, v[2] = hi.x, v[3] = hi.y;
-}
-
 template <typename TX, typename TW, typename TY, bool VEC>
 __global__ void __launch_bounds__(256, 2) linear_narrow_kernel(LinearArgs a) {
   __shared__ __align__(16) float nxs[kNarrowRows][kNarrowKC];
@@ -126,7 +116,7 @@ __global__ void __launch_bounds__(256, 2) linear_narrow_kernel(LinearArgs a) {
       for (int e = threadIdx.x; e < kNarrowRows * k4n; e += blockDim.x) {
         const int r = e / k4n, k = (e - r * k4n) << 2;
         float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (r < nr) nld4(X + (long long)(m0 + r) * a.ldx + kc + k, v);
+        if (r < nr) ld4(X + (long long)(m0 + r) * a.ldx + kc + k, v);
         *reinterpret_cast<float4*>(&nxs[r][k]) = make_float4(v[0], v[1], v[2], v[3]);
       }
     } else {
@@ -145,7 +135,7 @@ __global__ void __launch_bounds__(256, 2) linear_narrow_kernel(LinearArgs a) {
         for (int k = lane * 4; k < knp; k += 128) {
           float wv[4];
           if (VEC) {
-            nld4(wr + k, wv);
+            ld4(wr + k, wv);
           } else {
 #pragma unroll
             for (int j = 0; j < 4; ++j) wv[j] = k + j < kn ? ldf(wr + k + j) : 0.f;

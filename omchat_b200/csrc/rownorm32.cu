@@ -136,22 +136,6 @@ __global__ void __launch_bounds__(256) post_norm_residual_kernel(const float* __
 
 // out = act(gate) * up over the two halves of a stacked projection: z [rows, 2 * n] -> out [rows, n]; the arithmetic is fp32.
 // Four neighbouring columns per thread (8- or 16-byte accesses) when the rows are laid out for it, else one.
-__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
-  const float4 t = *reinterpret_cast<const float4*>(p);
-  v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
-}
-__device__ __forceinline__ void ld4(const bf16_t* p, float (&v)[4]) {
-  const uint2 t = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
-  v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
-}
-__device__ __forceinline__ void st4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-__device__ __forceinline__ void st4(bf16_t* p, const float (&v)[4]) {
-  uint2 t;
-  *reinterpret_cast<__nv_bfloat162*>(&t.x) = __floats2bfloat162_rn(v[0], v[1]);
-  *reinterpret_cast<__nv_bfloat162*>(&t.y) = __floats2bfloat162_rn(v[2], v[3]);
-  *reinterpret_cast<uint2*>(p) = t;
-}
 struct GluParams {
   int act;
   float limit, slope, shift;   // OMC_ACT_CLAMP_SWISH only

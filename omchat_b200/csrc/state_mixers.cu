@@ -15,6 +15,8 @@
 // two dot products of a token with three shuffles each. Tokens are staged 16 at a time in shared memory by cp.async, one chunk ahead of the one being
 // computed (decays, sigmoid and silu applied in place on arrival), so the sequential loop touches registers and shared memory only.
 // Recurrences whose channels carry one or a few states of their own (selective scan, gated linear recurrent unit) follow below.
+#include <type_traits>
+
 #include "seq_common.cuh"
 
 namespace omc {
@@ -90,6 +92,64 @@ __global__ void __launch_bounds__(256) causal_conv_silu_kernel(const float* __re
   }
 }
 
+// The convolution without unit vectors, four neighbouring channels per thread: a thread walks ROWS consecutive rows with the last
+// TAPS - 1 inputs in registers, so a row of x is read once per tile (plus TAPS - 1 rows in front of it), and nothing goes through
+// shared memory. Same sums in the same order as causal_conv_silu_kernel.
+template <typename TW, typename TY, int TAPS, int ROWS>
+__global__ void __launch_bounds__(128) causal_conv_rows_kernel(const float* __restrict__ x, long long ldx, int T, int ch,
+                                                               const TW* __restrict__ w, const TW* __restrict__ bias,
+                                                               const int32_t* __restrict__ pos, const int32_t* __restrict__ slot,
+                                                               float* __restrict__ state, TY* __restrict__ y, long long ldy, int save_here,
+                                                               int act) {
+  constexpr int R = TAPS - 1;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= ch) return;
+  const int t0 = blockIdx.x * ROWS, nr = min(ROWS, T - t0);
+  float wv[TAPS][4], b4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j][i] = ldf(w + (long long)(c + i) * TAPS + j);
+    if (bias != nullptr) b4[i] = ldf(bias + c + i);
+  }
+  float4 xv[ROWS], h[R > 0 ? R : 1];   // h[j]: the input R - j positions back
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) xv[r] = r < nr ? *reinterpret_cast<const float4*>(x + (long long)(t0 + r) * ldx + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  int prev = -1;   // slot of the row before
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    if (r < nr) {
+      const int t = t0 + r, s = slot[t], p = pos[t];
+      if (s != prev) {   // first row of the tile, or of another request: the inputs in front come from the step, the ring or are zero
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+          const int back = R - j, sp = p - back;
+          const float* q = nullptr;
+          if (sp >= 0) q = (t - back >= 0 && slot[t - back] == s) ? x + (long long)(t - back) * ldx : state + ((long long)s * R + sp % R) * ch;
+          h[j] = q != nullptr ? *reinterpret_cast<const float4*>(q + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        prev = s;
+      }
+      float o[4] = {b4[0], b4[1], b4[2], b4[3]};
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const float4 v = j < R ? h[j < R ? j : 0] : xv[r];
+        o[0] = fmaf(wv[j][0], v.x, o[0]), o[1] = fmaf(wv[j][1], v.y, o[1]), o[2] = fmaf(wv[j][2], v.z, o[2]), o[3] = fmaf(wv[j][3], v.w, o[3]);
+      }
+      if (act) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[i] = silu_f(o[i]);
+      }
+      st4(y + (long long)t * ldy + c, o);
+      // this thread is the only one that touches these channels of the ring: its write follows its reads
+      if (save_here && R > 0) *reinterpret_cast<float4*>(state + ((long long)s * R + p % (R > 0 ? R : 1)) * ch + c) = xv[r];
+#pragma unroll
+      for (int j = 0; j + 1 < R; ++j) h[j] = h[j + 1];
+      if (R > 0) h[R > 0 ? R - 1 : 0] = xv[r];
+    }
+  }
+}
+
 // The same convolution (no activation) in front of an attention: the first nq + nk channels are queries and keys that get an RMS norm
 // per `group` channels (a head, or one score map of a head) with the weights wq / wk [group]; queries go to q_out, normed keys and the
 // remaining channels (values) to the row of (slot, position) in the paged cache [pages][page_size][ch - nq]. One launch instead of
@@ -161,14 +221,24 @@ __global__ void __launch_bounds__(256) conv_qk_norm_store_kernel(const float* __
 // The last taps - 1 inputs of every request of the step go into its ring (rows that are followed by taps - 1 more rows of the
 // same request are not among them). A launch of its own when a request may have several rows: a row's ring entry is read by
 // CTAs of other rows of the convolution kernel.
+constexpr int kSaveRows = 64;   // rows a CTA looks through
 __global__ void __launch_bounds__(256) conv_state_save_kernel(const float* __restrict__ x, long long ldx, int ch, int R, int T,
                                                               const int32_t* __restrict__ pos, const int32_t* __restrict__ slot,
                                                               float* __restrict__ state) {
-  const int t = blockIdx.x;
-  const int s = slot[t];
-  if (t + R < T && slot[t + R] == s) return;
-  float* dst = state + ((long long)s * R + pos[t] % R) * ch;
-  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ch; c += gridDim.y * blockDim.x) dst[c] = x[(long long)t * ldx + c];
+  __shared__ int s_last[kSaveRows];
+  __shared__ int s_n;
+  if (threadIdx.x == 0) s_n = 0;
+  __syncthreads();
+  if (threadIdx.x < kSaveRows) {
+    const int t = blockIdx.x * kSaveRows + threadIdx.x;
+    if (t < T && !(t + R < T && slot[t + R] == slot[t])) s_last[atomicAdd(&s_n, 1)] = t;
+  }
+  __syncthreads();
+  for (int i = 0; i < s_n; ++i) {   // every (row, channel) has a ring entry of its own: the order does not matter
+    const int t = s_last[i];
+    float* dst = state + ((long long)slot[t] * R + pos[t] % R) * ch;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ch; c += gridDim.y * blockDim.x) dst[c] = x[(long long)t * ldx + c];
+  }
 }
 
 // ---- linear-state recurrence ----------------------------------------------------------------------------------------------
@@ -713,7 +783,7 @@ __global__ void __launch_bounds__(kSelThreads) selective_scan_kernel(SelArgs a) 
 // gets its start state and goes over its K tokens once more from registers. A run's whole decay is applied as expm1 of the summed
 // log a - never as a product of rounded decays - so the state keeps its digits however the tokens are spread over threads. The output
 // is multiplied by gelu of the other branch. FAST (bf16 operands): hardware exponential, reciprocal and square root.
-constexpr int kLruTok = 8;
+constexpr int kLruTok = 4;
 
 struct LruArgs {
   const void* u;
@@ -759,33 +829,43 @@ __global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
   const bool live = c < a.width;
   const int r0 = a.row_begin[blockIdx.y], r1 = a.row_begin[blockIdx.y + 1];
   if (r1 <= r0) return;
+  const int end = live ? r1 : r0;   // channels past the last take part in the barriers only
   const bool fresh = a.pos[r0] == 0;
   float* Sp = a.state + (long long)a.slot[r0] * a.width + c;
   float carry = (live && !fresh) ? *Sp : 0.f;
   const int blk = live ? c / a.n : 0, gr = blk * 2 * a.n + (live ? c - blk * a.n : 0), gi = gr + a.n;
   const float sp = live ? -a.scale * softplus_f(a.lam[c]) : 0.f;
   const float br = (live && a.gb != nullptr) ? a.gb[gr] : 0.f, bi = (live && a.gb != nullptr) ? a.gb[gi] : 0.f;
-  const TD* ug = static_cast<const TD*>(a.u);
-  TD* og = static_cast<TD*>(a.out);
+  const TD* ug = static_cast<const TD*>(a.u) + (live ? c : 0);
+  TD* og = static_cast<TD*>(a.out) + c;
+  float zr[K], zi[K], uv[K], yv[K];   // the raw inputs of this thread's next run
+  auto load = [&](int tb) {
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+      const long long t = tb + k;
+      const bool ok = tb + k < end;
+      zr[k] = ok ? a.g[t * a.ldg + gr] : 0.f;
+      zi[k] = ok ? a.g[t * a.ldg + gi] : 0.f;
+      uv[k] = ok ? ldf(ug + t * a.ldu) : 0.f;
+      yv[k] = (ok && a.y != nullptr) ? a.y[t * a.ldy + c] : 0.f;
+    }
+  };
+  load(r0 + wy * K);
   int buf = 0;
   for (int t0 = r0; t0 < r1; t0 += W * K, buf ^= 1) {
     const int tb = t0 + wy * K;
-    float am1[K], in[K], yv[K];
+    float am1[K], in[K], yc[K];
     float L = 0.f, loc = 0.f;
 #pragma unroll
     for (int k = 0; k < K; ++k) {
-      am1[k] = in[k] = yv[k] = 0.f;
-      const long long t = tb + k;
-      if (live && t < r1) {
-        const float zr = a.g[t * a.ldg + gr], zi = a.g[t * a.ldg + gi], uv = ldf(ug + t * a.ldu + c);
-        if (a.y != nullptr) yv[k] = a.y[t * a.ldy + c];
-        const float la = sp * lru_sigmoid<FAST>(zr + br);
-        am1[k] = lru_expm1<FAST>(la);
-        in[k] = lru_sqrt<FAST>(-am1[k] * (2.f + am1[k])) * (lru_sigmoid<FAST>(zi + bi) * uv);
-        L += la;
-        loc = fmaf(am1[k], loc, loc) + in[k];
-      }
+      const float la = tb + k < end ? sp * lru_sigmoid<FAST>(zr[k] + br) : 0.f;   // past the end: a = 1 and no input
+      am1[k] = lru_expm1<FAST>(la);
+      in[k] = lru_sqrt<FAST>(-am1[k] * (2.f + am1[k])) * (lru_sigmoid<FAST>(zi[k] + bi) * uv[k]);
+      yc[k] = yv[k];
+      L += la;
+      loc = fmaf(am1[k], loc, loc) + in[k];
     }
+    load(tb + W * K);   // on its way during the rest of this tile
     float S = carry;
     if (W > 1) {
       float2* run = s_run + (size_t)buf * W * CX;
@@ -799,10 +879,9 @@ __global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
     }
 #pragma unroll
     for (int k = 0; k < K; ++k) {
-      const long long t = tb + k;
-      if (live && t < r1) {
+      if (tb + k < end) {
         S = fmaf(am1[k], S, S) + in[k];
-        stf(og + t * a.ldo + c, a.y != nullptr ? S * lru_gelu<FAST>(yv[k]) : S);
+        stf(og + (long long)(tb + k) * a.ldo, a.y != nullptr ? S * lru_gelu<FAST>(yc[k]) : S);
       }
     }
     if (W == 1) carry = S;
@@ -823,6 +902,30 @@ extern "C" int omc_causal_conv(const float* x, long long ldx, int T, int ch, con
       (unit_channels > 0 && scaled_channels % unit_group))
     return set_error(OMC_ERR_ARG, "omc_causal_conv: bad argument");
   if (T == 0) return OMC_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool rows4 = unit_channels == 0 && taps <= 4 && ch % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0 &&
+                     reinterpret_cast<uintptr_t>(y) % 16 == 0 && (state == nullptr || reinterpret_cast<uintptr_t>(state) % 16 == 0);
+  if (rows4) {
+    const int b4 = (ch / 4 + 127) / 128;
+    if (b4 > 65535) return set_error(OMC_ERR_SHAPE, "omc_causal_conv: too many channel blocks");
+    OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(y_dt, TY, {
+      auto go = [&](auto taps_c) {
+        constexpr int TAPS = decltype(taps_c)::value;
+        if (T >= 256)
+          causal_conv_rows_kernel<TW, TY, TAPS, kConvRows><<<dim3((T + kConvRows - 1) / kConvRows, b4), 128, 0, st>>>(
+              x, ldx, T, ch, static_cast<const TW*>(w), static_cast<const TW*>(bias), pos, slot, state, static_cast<TY*>(y), ldy, single_rows ? 1 : 0, act == OMC_CONV_SILU ? 1 : 0);
+        else
+          causal_conv_rows_kernel<TW, TY, TAPS, 1><<<dim3(T, b4), 128, 0, st>>>(
+              x, ldx, T, ch, static_cast<const TW*>(w), static_cast<const TW*>(bias), pos, slot, state, static_cast<TY*>(y), ldy, single_rows ? 1 : 0, act == OMC_CONV_SILU ? 1 : 0);
+      };
+      if (taps == 1) go(std::integral_constant<int, 1>());
+      else if (taps == 2) go(std::integral_constant<int, 2>());
+      else if (taps == 3) go(std::integral_constant<int, 3>());
+      else go(std::integral_constant<int, 4>());
+    }))
+    if (taps > 1 && !single_rows) conv_state_save_kernel<<<dim3((T + kSaveRows - 1) / kSaveRows, (ch + 255) / 256), 256, 0, st>>>(x, ldx, ch, taps - 1, T, pos, slot, state);
+    return check_launch("omc_causal_conv");
+  }
   // channel blocks of about 512 channels, whole unit-vector groups each
   int ch_block = 512;
   if (unit_channels > 0) ch_block = unit_group >= 512 ? unit_group : (512 / unit_group) * unit_group;
@@ -830,7 +933,6 @@ extern "C" int omc_causal_conv(const float* x, long long ldx, int T, int ch, con
   if ((size_t)ch_block * kConvRows * sizeof(float) > 200 * 1024) return set_error(OMC_ERR_SHAPE, "omc_causal_conv: unit-vector group too wide for shared memory");
   const int blocks = (ch + ch_block - 1) / ch_block;
   if (blocks > 65535) return set_error(OMC_ERR_SHAPE, "omc_causal_conv: too many channel blocks");
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rows_per_cta = T >= 256 ? kConvRows : 1;   // short steps (decode) keep one CTA per row: there are few rows to share anything
   const size_t smem = (size_t)ch_block * rows_per_cta * sizeof(float);
   OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(y_dt, TY, {
@@ -839,7 +941,7 @@ extern "C" int omc_causal_conv(const float* x, long long ldx, int T, int ch, con
         x, ldx, T, ch, ch_block, rows_per_cta, static_cast<const TW*>(w), static_cast<const TW*>(bias), taps, pos, slot, state,
         static_cast<TY*>(y), ldy, unit_channels, unit_group, unit_eps, scaled_channels, unit_mult, single_rows ? 1 : 0, act == OMC_CONV_SILU ? 1 : 0);
   }))
-  if (taps > 1 && !single_rows) conv_state_save_kernel<<<dim3(T, (ch + 1023) / 1024), 256, 0, st>>>(x, ldx, ch, taps - 1, T, pos, slot, state);
+  if (taps > 1 && !single_rows) conv_state_save_kernel<<<dim3((T + kSaveRows - 1) / kSaveRows, (ch + 255) / 256), 256, 0, st>>>(x, ldx, ch, taps - 1, T, pos, slot, state);
   return check_launch("omc_causal_conv");
 }
 
@@ -867,7 +969,7 @@ extern "C" int omc_conv_qk_norm_kv_store(const float* x, long long ldx, int T, i
         static_cast<const TW*>(wk), eps, block_table, max_pages, page_size, static_cast<TC*>(pool), static_cast<TC*>(q_out), ldqo,
         single_rows ? 1 : 0);
   }))
-  if (taps > 1 && !single_rows) conv_state_save_kernel<<<dim3(T, (ch + 1023) / 1024), 256, 0, st>>>(x, ldx, ch, taps - 1, T, pos, slot, state);
+  if (taps > 1 && !single_rows) conv_state_save_kernel<<<dim3((T + kSaveRows - 1) / kSaveRows, (ch + 255) / 256), 256, 0, st>>>(x, ldx, ch, taps - 1, T, pos, slot, state);
   return check_launch("omc_conv_qk_norm_kv_store");
 }
 
@@ -1025,7 +1127,7 @@ static int launch_rglru(const LruArgs& a, int rows, int portions, cudaStream_t s
   if (avg <= 2) {
     rglru_scan_kernel<TD, FAST, 1><<<dim3((a.width + 127) / 128, portions), dim3(128, 1), 0, st>>>(a);
   } else {
-    const int W = avg >= 96 ? 16 : (avg >= 24 ? 4 : 2);
+    const int W = avg >= 48 ? 8 : (avg >= 12 ? 4 : 2);
     rglru_scan_kernel<TD, FAST, kLruTok><<<dim3((a.width + 31) / 32, portions), dim3(32, W), (size_t)2 * W * 32 * sizeof(float2), st>>>(a);
   }
   return check_launch("omc_rglru_scan");

@@ -54,7 +54,7 @@ class LatentAttention:
             if "portions" in plans:
                 plan = seqlib.LatentAttnPlan(plans["portions"], H, self.device, window=window)
             else:
-                parts = plans["decode_parts"] if "decode_parts" in plans else seqlib.DecodeAttnPlan.parts_for(T, min(window, plans["decode_keys"]))
+                parts = plans["decode_parts"] if "decode_parts" in plans else seqlib.DecodeAttnPlan.parts_for(T, min(window, plans["decode_keys"]), min_keys=64)
                 key = (T, H, parts, window)
                 plan = self._decode_plans.get(key)
                 if plan is None:
