@@ -787,16 +787,16 @@ constexpr int kLruTok = 4;
 
 struct LruArgs {
   const void* u;
-  long long ldu;
+  int ldu;
   const float* g;
-  long long ldg;
+  int ldg;
   const float* gb;
   const float* lam;
   const float* y;
-  long long ldy;
+  int ldy;
   float* state;
   void* out;
-  long long ldo;
+  int ldo;
   const int32_t* row_begin;
   const int32_t* pos;
   const int32_t* slot;
@@ -804,22 +804,41 @@ struct LruArgs {
   float scale;
 };
 
+__device__ __forceinline__ float ex2_approx(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
 template <bool FAST>
-__device__ __forceinline__ float lru_sigmoid(float z) { return FAST ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z); }
+__device__ __forceinline__ float lru_sigmoid(float z) {
+  return FAST ? rcp_approx(1.f + ex2_approx(-1.4426950408889634f * z)) : sigmoid_f(z);
+}
 template <bool FAST>
 __device__ __forceinline__ float lru_sqrt(float z) {
   if (!FAST) return sqrtf(z);
   float r;
-  asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(z));
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(z));
   return r;
 }
+// gelu in its tanh form: 0.5 z (1 + tanh(p)) = z sigmoid(2 p)
 template <bool FAST>
 __device__ __forceinline__ float lru_gelu(float z) {
   const float p = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
-  return 0.5f * z * (1.f + (FAST ? 1.f - __fdividef(2.f, __expf(2.f * p) + 1.f) : tanhf(p)));
+  return FAST ? z * lru_sigmoid<true>(2.f * p) : 0.5f * z * (1.f + tanhf(p));
 }
+// exp(x) - 1 for x <= 0 (FAST: expm1_decay_f with the hardware exponential as it is)
 template <bool FAST>
-__device__ __forceinline__ float lru_expm1(float x) { return FAST ? expm1_decay_f(x) : expm1f(x); }
+__device__ __forceinline__ float lru_expm1(float x) {
+  if (!FAST) return expm1f(x);
+  const float p = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  const float e = ex2_approx(x * 1.4426950408889634f) - 1.f;
+  return x > -0.1f ? p : e;
+}
 
 template <typename TD, bool FAST, int K>
 __global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
@@ -829,25 +848,27 @@ __global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
   const bool live = c < a.width;
   const int r0 = a.row_begin[blockIdx.y], r1 = a.row_begin[blockIdx.y + 1];
   if (r1 <= r0) return;
-  const int end = live ? r1 : r0;   // channels past the last take part in the barriers only
+  const int end = live ? r1 : r0, last = r1 - 1;   // channels past the last read channel 0 and take part in the barriers only
   const bool fresh = a.pos[r0] == 0;
   float* Sp = a.state + (long long)a.slot[r0] * a.width + c;
   float carry = (live && !fresh) ? *Sp : 0.f;
-  const int blk = live ? c / a.n : 0, gr = blk * 2 * a.n + (live ? c - blk * a.n : 0), gi = gr + a.n;
+  const int blk = live ? c / a.n : 0, gr = blk * 2 * a.n + (live ? c - blk * a.n : 0);
   const float sp = live ? -a.scale * softplus_f(a.lam[c]) : 0.f;
-  const float br = (live && a.gb != nullptr) ? a.gb[gr] : 0.f, bi = (live && a.gb != nullptr) ? a.gb[gi] : 0.f;
-  const TD* ug = static_cast<const TD*>(a.u) + (live ? c : 0);
-  TD* og = static_cast<TD*>(a.out) + c;
+  const float br = (live && a.gb != nullptr) ? a.gb[gr] : 0.f, bi = (live && a.gb != nullptr) ? a.gb[gr + a.n] : 0.f;
+  const TD* ug = static_cast<const TD*>(a.u) + (long long)r0 * a.ldu + (live ? c : 0);
+  const float* pr = a.g + (long long)r0 * a.ldg + gr;
+  const float* pi = pr + a.n;
+  const float* yg = a.y != nullptr ? a.y + (long long)r0 * a.ldy + (live ? c : 0) : nullptr;
+  TD* og = static_cast<TD*>(a.out) + (long long)r0 * a.ldo + c;
   float zr[K], zi[K], uv[K], yv[K];   // the raw inputs of this thread's next run
   auto load = [&](int tb) {
 #pragma unroll
     for (int k = 0; k < K; ++k) {
-      const long long t = tb + k;
-      const bool ok = tb + k < end;
-      zr[k] = ok ? a.g[t * a.ldg + gr] : 0.f;
-      zi[k] = ok ? a.g[t * a.ldg + gi] : 0.f;
-      uv[k] = ok ? ldf(ug + t * a.ldu) : 0.f;
-      yv[k] = (ok && a.y != nullptr) ? a.y[t * a.ldy + c] : 0.f;
+      const int t = min(tb + k, last) - r0;   // past the end: read the last row, whose copy contributes nothing below
+      zr[k] = pr[(long long)t * a.ldg];
+      zi[k] = pi[(long long)t * a.ldg];
+      uv[k] = ldf(ug + (long long)t * a.ldu);
+      yv[k] = yg != nullptr ? yg[(long long)t * a.ldy] : 0.f;
     }
   };
   load(r0 + wy * K);
@@ -881,7 +902,7 @@ __global__ void __launch_bounds__(512) rglru_scan_kernel(LruArgs a) {
     for (int k = 0; k < K; ++k) {
       if (tb + k < end) {
         S = fmaf(am1[k], S, S) + in[k];
-        stf(og + (long long)(tb + k) * a.ldo, a.y != nullptr ? S * lru_gelu<FAST>(yc[k]) : S);
+        stf(og + (long long)(tb + k - r0) * a.ldo, yg != nullptr ? S * lru_gelu<FAST>(yc[k]) : S);
       }
     }
     if (W == 1) carry = S;
@@ -1127,7 +1148,7 @@ static int launch_rglru(const LruArgs& a, int rows, int portions, cudaStream_t s
   if (avg <= 2) {
     rglru_scan_kernel<TD, FAST, 1><<<dim3((a.width + 127) / 128, portions), dim3(128, 1), 0, st>>>(a);
   } else {
-    const int W = avg >= 48 ? 8 : (avg >= 12 ? 4 : 2);
+    const int W = avg >= 96 ? 16 : (avg >= 24 ? 8 : (avg >= 12 ? 4 : 2));
     rglru_scan_kernel<TD, FAST, kLruTok><<<dim3((a.width + 31) / 32, portions), dim3(32, W), (size_t)2 * W * 32 * sizeof(float2), st>>>(a);
   }
   return check_launch("omc_rglru_scan");
@@ -1141,7 +1162,8 @@ extern "C" int omc_rglru_scan(const void* u, int dt, long long ldu, const float*
     return set_error(OMC_ERR_ARG, "omc_rglru_scan: bad argument");
   if (portions == 0) return OMC_OK;
   if (portions > 65535) return set_error(OMC_ERR_SHAPE, "omc_rglru_scan: more than 65535 portions");
-  const LruArgs a{u, ldu, g, ldg, gb, lam, y, ldy, state, out, ldo, row_begin, pos, slot, width, width / blocks, decay_scale};
+  if (ldu > INT32_MAX || ldg > INT32_MAX || ldy > INT32_MAX || ldo > INT32_MAX) return set_error(OMC_ERR_SHAPE, "omc_rglru_scan: row stride above 2^31");
+  const LruArgs a{u, (int)ldu, g, (int)ldg, gb, lam, y, (int)ldy, state, out, (int)ldo, row_begin, pos, slot, width, width / blocks, decay_scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (dt == OMC_DT_F32) return launch_rglru<float, false>(a, rows, portions, st);
   if (dt == OMC_DT_BF16) return launch_rglru<bf16_t, true>(a, rows, portions, st);

@@ -33,7 +33,7 @@ from .. import lib, seqlib
 from ..config import ClampedMlpSpec, GatedLruSpec, GroupedMoeSpec, LatentAttentionSpec, MunevikConfig
 from .paged_cache import PagedStateCache
 from .seq_latent import LatentAttention
-from .seq_linear import dense_linear, stack_rows
+from .seq_linear import NARROW_GEMM_MIN_WEIGHT, dense_linear, stack_rows
 from .seq_model import GraphedDecodeMixin, SequenceStepLM, portion_starts
 from .seq_moe import expert_workspace, grouped_tensor_gemm_ok, run_sorted_experts
 
@@ -249,8 +249,10 @@ class MunevikDecoder(GraphedDecodeMixin):
         wins = [l.mixer.window or seqlib.WINDOW_ALL for l in self.cfg.layers if isinstance(l.mixer, LatentAttentionSpec)]
         return {"decode_keys": 1 << max(min(max(wins, default=1), max_keys) - 1, 0).bit_length()}
 
-    def _linear(self, x, w, out_dtype, bias=None):
-        return dense_linear(x, w, out_dtype, tensor_gemm=self.tensor_gemm, bias=bias)
+    def _linear(self, x, w, out_dtype, bias=None, narrow: bool = False):
+        """narrow: few outputs over a long K (router, head gates): on long steps the tensor-core GEMM takes it from a much smaller
+        matrix on than the general rule says."""
+        return dense_linear(x, w, out_dtype, tensor_gemm=self.tensor_gemm, bias=bias, min_weight=NARROW_GEMM_MIN_WEIGHT if narrow else None)
 
     def _one_product(self, T: int) -> bool:
         """Short steps pay per launch: one fp32 product over all rows of a stacked matrix. Long steps pay per byte: what feeds another
@@ -270,7 +272,7 @@ class MunevikDecoder(GraphedDecodeMixin):
             if self.dtype != f32:   # the unrotated queries are operands of the absorbing product
                 qn = torch.empty(T, H * dn, device=dev, dtype=self.dtype)
         else:
-            q, z, off = self._linear(xb, mw.w_in[:mw.nq], self.dtype), self._linear(xb, mw.w_in[mw.nq:], f32), mw.nq
+            q, z, off = self._linear(xb, mw.w_in[:mw.nq], self.dtype), self._linear(xb, mw.w_in[mw.nq:], f32, narrow=True), mw.nq
         gate = z[:, mw.cols["g"].start - off:mw.cols["g"].stop - off]
         dkv = z[:, mw.cols["dkv"].start - off:mw.cols["dkv"].stop - off] if own else None
         pool = cache.pools[li if own else m.kv_from]
@@ -314,10 +316,10 @@ class MunevikDecoder(GraphedDecodeMixin):
         tile = 128 if grouped else seqlib.LINEAR_TILE
         ws = expert_workspace(self._moe_ws, T, s.experts, s.top, s.expert_ff, tile, self.C, self.dtype, self.device)
         if self._one_product(T) or not s.shared_ff:
-            z = self._linear(xb, mw.w_in, f32)
+            z = self._linear(xb, mw.w_in, f32, narrow=True)
             zs = z[:, mw.n_router:]
         else:
-            z, zs = self._linear(xb, mw.w_in[:mw.n_router], f32), self._linear(xb, mw.w_in[mw.n_router:], self.dtype)
+            z, zs = self._linear(xb, mw.w_in[:mw.n_router], f32, narrow=True), self._linear(xb, mw.w_in[mw.n_router:], self.dtype)
         seqlib.router_topk(z, s.experts, s.experts, s.top, None, False, ws.ids, ws.w, None, ws.counts, score=seqlib.ROUTER_SIGMOID, groups=s.groups,
                            keep=s.keep, scale=s.scale)
         run_sorted_experts(ws, xb, s.experts, s.top, s.expert_ff, tile, mw.gate_up, mw.down, seqlib.ACT_SILU, grouped=grouped)

@@ -54,7 +54,7 @@ class LatentAttention:
             if "portions" in plans:
                 plan = seqlib.LatentAttnPlan(plans["portions"], H, self.device, window=window)
             else:
-                parts = plans["decode_parts"] if "decode_parts" in plans else seqlib.DecodeAttnPlan.parts_for(T, min(window, plans["decode_keys"]), min_keys=64)
+                parts = plans["decode_parts"] if "decode_parts" in plans else self._decode_parts(T, min(window, plans["decode_keys"]))
                 key = (T, H, parts, window)
                 plan = self._decode_plans.get(key)
                 if plan is None:
@@ -62,6 +62,12 @@ class LatentAttention:
                 plan.fill(pos, slot)
             plans[(H, window)] = plan
         return plan
+
+    @staticmethod
+    def _decode_parts(T: int, keys: int) -> int:
+        """Key ranges per row of a decode-only step: of 128 keys or more, of 64 where a short window would leave SMs without a CTA."""
+        parts = seqlib.DecodeAttnPlan.parts_for(T, keys)
+        return parts if T * parts >= 148 else seqlib.DecodeAttnPlan.parts_for(T, keys, min_keys=64)
 
     def attend(self, qcat: torch.Tensor, r: int, dr: int, pool: torch.Tensor, cache, pos, slot, plans: Optional[dict], scale: float, *,
                sink: Optional[torch.Tensor] = None, window: Optional[int] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -18,6 +18,7 @@ from .. import lib, seqlib
 
 TENSOR_GEMM_MIN_WEIGHT = 1 << 20
 SKINNY_GEMM_MIN_WEIGHT = 1 << 17
+NARROW_GEMM_MIN_WEIGHT = 1 << 15   # min_weight for narrow products (routers, gates, low-rank factors) of a design that asks for it
 _TENSOR_EPILOGUES = {seqlib.ACT_RELU2: lib.EPI_RELU2, seqlib.ACT_GELU_ERF: lib.EPI_GELU}   # activations the tensor-core GEMMs apply themselves
 
 

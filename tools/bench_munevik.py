@@ -33,6 +33,7 @@ import torch  # noqa: E402
 from omchat_b200 import seqlib  # noqa: E402
 from omchat_b200.config import MunevikConfig, VoduzenConfig  # noqa: E402
 from omchat_b200.model import munevik, voduzen  # noqa: E402
+from omchat_b200.model.seq_latent import LatentAttention  # noqa: E402
 from tools.bench_fofisun import serve  # noqa: E402
 from tools.bench_voduzen import peaks, timed  # noqa: E402
 
@@ -188,7 +189,7 @@ def kernels(z, n_seq, L, B, ctx):
     for name, win, gt in (("voduzen_latent_attn_decode", seqlib.WINDOW_ALL, None), ("latent_attn_window_gate_decode", z["win"], gate[:B]),
                           ("latent_attn_window256_gate_decode", 256, gate[:B])):
         keys = min(win, ctx + 1)
-        plan = seqlib.DecodeAttnPlan(B, H, seqlib.DecodeAttnPlan.parts_for(B, keys), dev, window=win)
+        plan = seqlib.DecodeAttnPlan(B, H, LatentAttention._decode_parts(B, keys), dev, window=win)
         plan.fill(posd, slotd)
         ms = timed(lambda: seqlib.latent_attn_mma(q, r, dr, pool, table, page, plan, None, 0.07, o, window=win, gate=gt))
         out[name] = rate(ms, B * keys * D * 2, batch=B, keys=keys, ctas=plan.n_items)
