@@ -170,9 +170,10 @@ int omc_post_norm_residual(const float* y1, long long ld1, const void* wa, const
 
 /* y[t, c] = act(z[t, c]) * z[t, n + c] for c < n: the two halves of a stacked gate | up projection. z of z_dt, fp32 arithmetic.
  * act OMC_ACT_CLAMP_SWISH: g = min(z[t, c], limit), u = clamp(z[t, n + c], -limit, limit), y = g * sigmoid(slope * g) * (u + shift);
- * limit, slope and shift are ignored by the other activations. */
+ * limit, slope and shift are ignored by the other activations. tile_group (NULL: all rows): rows of tiles with tile_group[t / tile]
+ * < 0 are skipped (tiles of the expert-sorted layout that hold no rows). */
 int omc_glu_mul(const void* z, int z_dt, long long ldz, int rows, int n, int act, float limit, float slope, float shift, void* y,
-                int y_dt, long long ldy, void* stream);
+                int y_dt, long long ldy, const int32_t* tile_group, int tile, void* stream);
 
 /* h32[t, :] = table[ids[t], :] * scale + s(pos[t]) with the sinusoidal position vector s(p)[2i] = sin(p * freq[i]),
  * s(p)[2i + 1] = cos(p * freq[i]); freq is a device table of ceil(C / 2) doubles (the angle is formed and reduced in double precision).

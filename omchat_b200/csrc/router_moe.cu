@@ -120,26 +120,56 @@ __global__ void __launch_bounds__(kRouteWarps * 32) router_topk_kernel(const flo
   if (has_gate && lane == 0) gate[t] = 1.f / (1.f + expf(-zr[E_tot]));
 }
 
+// Segment starts (whole tiles) and the tile -> expert table by the calling warp, 32 experts at a time; next (NULL to skip) receives
+// every segment's first row too. counts are left zeroed.
+__device__ __forceinline__ void plan_segments(int32_t* counts, int experts, int tile, int max_tiles, int32_t* seg_start, int32_t* tile_group,
+                                              int32_t* next) {
+  const int lane = threadIdx.x & 31;
+  int tiles = 0;
+  for (int e0 = 0; e0 < experts; e0 += 32) {
+    const int e = e0 + lane;
+    const int n = e < experts ? (counts[e] + tile - 1) / tile : 0;
+    int incl = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    const int first = tiles + incl - n;
+    if (e < experts) {
+      seg_start[e] = first * tile;
+      if (next != nullptr) next[e] = first * tile;
+      counts[e] = 0;
+      for (int i = 0; i < n && first + i < max_tiles; ++i) tile_group[first + i] = e;
+    }
+    tiles += __shfl_sync(0xffffffffu, incl, 31);
+  }
+  if (lane == 0) seg_start[experts] = tiles * tile;
+}
+
 __global__ void __launch_bounds__(256) moe_plan_tiles_kernel(int32_t* __restrict__ counts, int experts, int tile, int max_tiles,
                                                              int32_t* __restrict__ seg_start, int32_t* __restrict__ cursor,
                                                              int32_t* __restrict__ tile_group) {
   for (int i = threadIdx.x; i < max_tiles; i += blockDim.x) tile_group[i] = -1;
+  for (int e = threadIdx.x; e < experts; e += blockDim.x) cursor[e] = 0;
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int tiles = 0;
-    for (int e = 0; e < experts; ++e) {
-      const int n = (counts[e] + tile - 1) / tile;
-      seg_start[e] = tiles * tile;
-      for (int i = 0; i < n && tiles + i < max_tiles; ++i) tile_group[tiles + i] = e;
-      tiles += n;
-    }
-    seg_start[experts] = tiles * tile;
+  if (threadIdx.x < 32) plan_segments(counts, experts, tile, max_tiles, seg_start, tile_group, nullptr);
+}
+
+// A row's copy into a segment: 16-byte pieces where both rows are laid out for them.
+template <typename TT>
+__device__ __forceinline__ void copy_row(const TT* src, TT* dst, int C, bool vec) {
+  if (vec) {
+    const int per = C * (int)sizeof(TT) / 16;
+    for (int i = threadIdx.x; i < per; i += blockDim.x) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+  } else {
+    for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = src[c];
   }
-  __syncthreads();
-  for (int e = threadIdx.x; e < experts; e += blockDim.x) {
-    counts[e] = 0;
-    cursor[e] = 0;
-  }
+}
+template <typename TT>
+__device__ __forceinline__ bool rows_in_16(const TT* x, long long ldx, const TT* xs, long long ldxs, int C) {
+  return ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xs) | (uintptr_t)(ldx * sizeof(TT)) | (uintptr_t)(ldxs * sizeof(TT)) |
+           (uintptr_t)(C * sizeof(TT))) & 15) == 0;
 }
 
 template <typename TT>
@@ -158,6 +188,7 @@ __global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const TT* __restr
     slot_of[(long long)t * top + threadIdx.x] = sl;
   }
   __syncthreads();
+  const bool vec = rows_in_16(x, ldx, xs, ldxs, C);
   for (int k = 0; k < top; ++k) {
     const int sl = s_slot[k];
     if (sl < 0) continue;
@@ -165,7 +196,7 @@ __global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const TT* __restr
       const float wk = row_w[(long long)t * top + k];
       for (int c = threadIdx.x; c < C; c += blockDim.x) stf(xs + (long long)sl * ldxs + c, wk * ldf(x + (long long)t * ldx + c));
     } else {
-      for (int c = threadIdx.x; c < C; c += blockDim.x) xs[(long long)sl * ldxs + c] = x[(long long)t * ldx + c];
+      copy_row(x + (long long)t * ldx, xs + (long long)sl * ldxs, C, vec);
     }
   }
 }
@@ -183,19 +214,9 @@ __global__ void __launch_bounds__(256) moe_plan_scatter_small_kernel(int32_t* __
   __shared__ int s_slot[32];
   for (int i = threadIdx.x; i < max_tiles; i += blockDim.x) tile_group[i] = -1;
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int tiles = 0;
-    for (int e = 0; e < experts; ++e) {
-      const int n = (counts[e] + tile - 1) / tile;
-      seg_start[e] = tiles * tile;
-      s_seg[e] = tiles * tile;
-      for (int i = 0; i < n && tiles + i < max_tiles; ++i) tile_group[tiles + i] = e;
-      tiles += n;
-      counts[e] = 0;
-    }
-    seg_start[experts] = tiles * tile;
-  }
+  if (threadIdx.x < 32) plan_segments(counts, experts, tile, max_tiles, seg_start, tile_group, s_seg);
   __syncthreads();
+  const bool vec = rows_in_16(x, ldx, xs, ldxs, C);
   for (int t = 0; t < T; ++t) {
     if (threadIdx.x == 0) {
       for (int k = 0; k < top; ++k) {
@@ -213,7 +234,7 @@ __global__ void __launch_bounds__(256) moe_plan_scatter_small_kernel(int32_t* __
       if (row_w != nullptr) {
         for (int c = threadIdx.x; c < C; c += blockDim.x) stf(xs + (long long)sl * ldxs + c, wk * ldf(x + (long long)t * ldx + c));
       } else {
-        for (int c = threadIdx.x; c < C; c += blockDim.x) xs[(long long)sl * ldxs + c] = x[(long long)t * ldx + c];
+        copy_row(x + (long long)t * ldx, xs + (long long)sl * ldxs, C, vec);
       }
     }
     __syncthreads();

@@ -155,12 +155,13 @@ __device__ __forceinline__ float glu_pair(float g, float u, const GluParams& p) 
 
 template <typename TZ, typename TY, int VEC>
 __global__ void __launch_bounds__(256) glu_mul_kernel(const TZ* __restrict__ z, long long ldz, int n, GluParams gp, TY* __restrict__ y,
-                                                      long long ldy, long long total) {
+                                                      long long ldy, long long total, const int32_t* __restrict__ tile_group, int tile) {
   const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;   // one thread per VEC columns
   if (e >= total) return;
   const int per_row = n / VEC;
   const long long t = e / per_row;
   const int c = (int)(e - t * per_row) * VEC;
+  if (tile_group != nullptr && tile_group[t / tile] < 0) return;   // a tile of the expert-sorted layout that no expert uses
   if (VEC == 4) {
     float g[4], u[4];
     ld4(z + t * ldz + c, g);
@@ -410,16 +411,16 @@ extern "C" int omc_post_norm_residual(const float* y1, long long ld1, const void
 }
 
 extern "C" int omc_glu_mul(const void* z, int z_dt, long long ldz, int rows, int n, int act, float limit, float slope, float shift,
-                           void* y, int y_dt, long long ldy, void* stream) {
-  if (z == nullptr || y == nullptr || rows < 0 || n <= 0) return set_error(OMC_ERR_ARG, "omc_glu_mul: bad argument");
+                           void* y, int y_dt, long long ldy, const int32_t* tile_group, int tile, void* stream) {
+  if (z == nullptr || y == nullptr || rows < 0 || n <= 0 || (tile_group != nullptr && tile <= 0)) return set_error(OMC_ERR_ARG, "omc_glu_mul: bad argument");
   if (rows == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const long long total = (long long)rows * n;
   const bool vec = n % 4 == 0 && ldz % 4 == 0 && ldy % 4 == 0 && reinterpret_cast<uintptr_t>(z) % 16 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0;
   const GluParams gp{act, limit, slope, shift};
   OMC_DT_SWITCH(z_dt, TZ, OMC_DT_SWITCH(y_dt, TY, {
-    if (vec) glu_mul_kernel<TZ, TY, 4><<<(unsigned)((total / 4 + 255) / 256), 256, 0, st>>>(static_cast<const TZ*>(z), ldz, n, gp, static_cast<TY*>(y), ldy, total / 4);
-    else glu_mul_kernel<TZ, TY, 1><<<(unsigned)((total + 255) / 256), 256, 0, st>>>(static_cast<const TZ*>(z), ldz, n, gp, static_cast<TY*>(y), ldy, total);
+    if (vec) glu_mul_kernel<TZ, TY, 4><<<(unsigned)((total / 4 + 255) / 256), 256, 0, st>>>(static_cast<const TZ*>(z), ldz, n, gp, static_cast<TY*>(y), ldy, total / 4, tile_group, tile);
+    else glu_mul_kernel<TZ, TY, 1><<<(unsigned)((total + 255) / 256), 256, 0, st>>>(static_cast<const TZ*>(z), ldz, n, gp, static_cast<TY*>(y), ldy, total, tile_group, tile);
   }))
   return check_launch("omc_glu_mul");
 }

@@ -783,7 +783,7 @@ __global__ void __launch_bounds__(kSelThreads) selective_scan_kernel(SelArgs a) 
 // gets its start state and goes over its K tokens once more from registers. A run's whole decay is applied as expm1 of the summed
 // log a - never as a product of rounded decays - so the state keeps its digits however the tokens are spread over threads. The output
 // is multiplied by gelu of the other branch. FAST (bf16 operands): hardware exponential, reciprocal and square root.
-constexpr int kLruTok = 4;
+constexpr int kLruTok = 4, kLruSms = 148;
 
 struct LruArgs {
   const void* u;
@@ -1148,7 +1148,8 @@ static int launch_rglru(const LruArgs& a, int rows, int portions, cudaStream_t s
   if (avg <= 2) {
     rglru_scan_kernel<TD, FAST, 1><<<dim3((a.width + 127) / 128, portions), dim3(128, 1), 0, st>>>(a);
   } else {
-    const int W = avg >= 96 ? 16 : (avg >= 24 ? 8 : (avg >= 12 ? 4 : 2));
+    int W = avg >= 96 ? 16 : (avg >= 24 ? 8 : (avg >= 12 ? 4 : 2));
+    if (W == 16 && (long long)((a.width + 31) / 32) * portions > 2 * kLruSms) W = 8;   // 16 runs fit an SM twice: no second wave for a few CTAs
     rglru_scan_kernel<TD, FAST, kLruTok><<<dim3((a.width + 31) / 32, portions), dim3(32, W), (size_t)2 * W * 32 * sizeof(float2), st>>>(a);
   }
   return check_launch("omc_rglru_scan");

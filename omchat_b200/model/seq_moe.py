@@ -73,7 +73,7 @@ def run_sorted_experts(ws: ExpertWorkspace, xb: torch.Tensor, experts: int, top:
         lib.gemm_grouped(ws.xs[:rows], gate_up, ws.tile_group, ws.gu[:rows], lib.EPI_NONE, hint)
     else:
         seqlib.linear(ws.xs, gate_up, ws.gu, M=rows, N=2 * ff, K=C, ldw=C, tile_group=ws.tile_group, group_stride=2 * ff * C)
-    seqlib.glu_mul(ws.gu[:rows], ff, act, ws.act[:rows], limit=limit, slope=slope, shift=shift)
+    seqlib.glu_mul(ws.gu[:rows], ff, act, ws.act[:rows], limit=limit, slope=slope, shift=shift, tile_group=ws.tile_group, tile=tile)
     if grouped:
         lib.gemm_grouped(ws.act[:rows], down, ws.tile_group, ws.ys[:rows], lib.EPI_NONE, hint)
     else:

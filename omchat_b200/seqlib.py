@@ -27,7 +27,7 @@ SIGNATURES = {
     "omc_linear": (_I, [_P, _I, _L, _L, _P, _I, _L, _L, _P, _I, _L, _L, _I, _I, _I, _I, _F, _I, _P, _L, _P]),
     "omc_linear_bias": (_I, [_P, _I, _L, _L, _P, _I, _L, _L, _P, _I, _L, _L, _I, _I, _I, _I, _F, _I, _P, _L, _P, _L, _P]),
     "omc_post_norm_residual": (_I, [_P, _L, _P, _P, _L, _P, _P, _I, _F, _F, _P, _L, _P, _P, _I, _L, _I, _I, _P]),
-    "omc_glu_mul": (_I, [_P, _I, _L, _I, _I, _I, _F, _F, _F, _P, _I, _L, _P]),
+    "omc_glu_mul": (_I, [_P, _I, _L, _I, _I, _I, _F, _F, _F, _P, _I, _L, _P, _I, _P]),
     "omc_embed_sinusoid": (_I, [_P, _P, _I, _P, _I, _I, _I, _F, _P, _P, _L, _P]),
     "omc_diff_heads_gate": (_I, [_P, _L, _I, _I, _I, _F, _F, _F, _P, _L, _I, _P, _I, _L, _P]),
     "omc_causal_conv": (_I, [_P, _L, _I, _I, _P, _P, _I, _I, _P, _P, _P, _P, _I, _L, _I, _I, _I, _F, _I, _F, _I, _P]),
@@ -451,13 +451,14 @@ def ln_residual(x: torch.Tensor, alpha: float, nw: torch.Tensor, nb: torch.Tenso
     return x_out if xb is None else xb
 
 
-def glu_mul(z: torch.Tensor, n: int, act: int, out: torch.Tensor, limit: float = 0.0, slope: float = 1.0, shift: float = 0.0):
+def glu_mul(z: torch.Tensor, n: int, act: int, out: torch.Tensor, limit: float = 0.0, slope: float = 1.0, shift: float = 0.0,
+            tile_group: Optional[torch.Tensor] = None, tile: int = 0):
     """out[:, c] = act(z[:, c]) * z[:, n + c]. ACT_CLAMP_SWISH: g = min(z[:, c], limit), u = clamp(z[:, n + c], -limit, limit),
-    out = g * sigmoid(slope * g) * (u + shift)."""
-    _need_cuda(z, out)
+    out = g * sigmoid(slope * g) * (u + shift). tile_group: rows of `tile`-row tiles that no expert uses are skipped."""
+    _need_cuda(z, out, tile_group)
     assert z.stride(1) == 1 and out.stride(1) == 1 and z.shape[1] >= 2 * n
     rc = load().omc_glu_mul(_ptr(z), _dt(z), z.stride(0), z.shape[0], n, act, limit, slope, shift, _ptr(out), _dt(out), out.stride(0),
-                            _stream())
+                            _ptr(tile_group), tile, _stream())
     _check(rc, "omc_glu_mul")
     return out
 
