@@ -64,9 +64,10 @@ int omc_latent_kv_store(const float* dkv, long long ld, int T, int r, int dr, co
                         int page_size, void* pool, int pool_dt, void* stream);
 
 /* omc_latent_kv_store and omc_rotary_q in one launch; w, pool and qcat share the dtype dt, q is of q_dt. dkv NULL: only the queries
- * (a layer that attends to another layer's cached rows). qn != NULL (dtype dt): receives the unrotated query parts, [T][H * dn]. */
+ * (a layer that attends to another layer's cached rows). qn != NULL (dtype dt): receives the unrotated query parts, [T][H * dn].
+ * rot_halves: dimension i of a rotated part is paired with i + rot_dims / 2 instead of 2i with 2i + 1. */
 int omc_latent_rope_store(const float* dkv, long long ld, int T, int r, int dr, const void* w, float eps, const float* cs, int rot_dims,
-                          const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size, void* pool,
+                          int rot_halves, const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size, void* pool,
                           const void* q, int q_dt, long long ldq, int H, int dn, void* qcat, void* qn, int dt, void* stream);
 
 /* Rotated query parts: q [T, H * (dn + dr)] of in_dt (per head dn unrotated then dr rotated dims) -> qcat[t][h][r + j] for
@@ -158,6 +159,12 @@ int omc_linear_bias(const void* X, int x_dt, long long ldx, long long sx, const 
                     void* Y, int y_dt, long long ldy, long long sy, int M, int N, int K, int batch, float alpha, int act,
                     const int32_t* tile_group, long long group_stride, const void* bias, long long sbias, void* stream);
 
+/* omc_linear (without a tile table) whose outputs are multiplied by a sigmoid gate: Y[b][m, n] = act(alpha * X W^T) * sigmoid(gate[m, b * sg + n]),
+ * gate rows of gate_dt at stride ldg (a column slice of another projection is fine). */
+int omc_linear_gate(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw, long long sw, void* Y, int y_dt,
+                    long long ldy, long long sy, int M, int N, int K, int batch, float alpha, int act, const void* gate, int gate_dt,
+                    long long ldg, long long sg, void* stream);
+
 /* Sublayer output -> residual stream -> next sublayer's input in one pass over the row:
  *   y = y1, or with y2 != NULL the mean of two branches, each normed with a plain weight first:
  *       y = (y1 / rms(y1) * wa + y2 / rms(y2) * wb) / 2
@@ -242,13 +249,14 @@ int omc_conv_qk_norm_kv_store(const float* x, long long ldx, int T, int ch, cons
  * decay_mode 0: g = decay_const[head]; 1: g = exp(-exp(A_log[head]) softplus(a[t, head] + dt_bias[head])); 2: one decay per key
  * channel, a [T, H * dim], dt_bias [H * dim]; 3: a [T, H * dim] holds the decays themselves; 4: g = sigmoid(a + dt_bias)^decay_pow per
  * key channel (dt_bias [H * dim] or NULL); 5: a holds g - 1. Modes 4 and 5 apply the decay as S + (g - 1) S, which keeps the digits
- * of a decay close to 1. The read-out is multiplied by out_scale (a query scale). beta raw [T, H], squashed by a sigmoid here. silu_in: q, k, v pass silu first.
+ * of a decay close to 1. 6 (state-space form): dt = softplus(a[t, head] + dt_bias[head]), g = exp(-exp(A_log[head]) dt), u_t = dt v_t and
+ * o_t = S^T q_t + D[head] v_t (D fp32 [H] or NULL; no beta), the decay applied as S + expm1(.) S. The read-out is multiplied by out_scale (a query scale). beta raw [T, H], squashed by a sigmoid here. silu_in: q, k, v pass silu first.
  * q / k [T, G * dim] (head h reads group h / (H / G)), v [T, H * vdim], out fp32 [T, H * vdim]. Portion i is rows
  * row_begin[i] .. row_begin[i + 1] - 1 (device int32 [portions + 1]), all of slot[row_begin[i]]; a portion whose first row has
  * position 0 starts from S = 0. Tokens are processed one after the other in every case. dim <= 256. */
 int omc_linear_state_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, int silu_in,
                           int decay_mode, const float* decay_const, const float* a, long long lda, const float* A_log,
-                          const float* dt_bias, const float* beta, long long ldb, float* state, float* out, long long ldo,
+                          const float* dt_bias, const float* D, const float* beta, long long ldb, float* state, float* out, long long ldo,
                           const int32_t* row_begin, int portions, const int32_t* pos, const int32_t* slot, int H, int G, int dim,
                           int vdim, float decay_pow, float out_scale, void* stream);
 
@@ -257,27 +265,36 @@ int omc_linear_state_scan(const float* q, long long ldq, const float* k, long lo
 int omc_gated_rms_rows(const float* x, long long ldx, int rows, int groups, int n, const void* w, int w_dt, float eps,
                        const float* gate, long long ldg, int gate_act, void* y, int y_dt, long long ldy, void* stream);
 
+/* The gate in front of the norm: v = x[t, :] * act(gate[t, :]), y[t, g * n + c] = v / sqrt(mean over part g of v^2 + eps) * w[g * n + c]
+ * for g < groups. gate of gate_dt, gate_act as above, w [groups * n] of w_dt, y of y_dt. */
+int omc_gate_rms_rows(const float* x, long long ldx, int rows, int groups, int n, const void* w, int w_dt, float eps, const void* gate,
+                      int gate_dt, long long ldg, int gate_act, void* y, int y_dt, long long ldy, void* stream);
+
 /* Rows of a step for windowed attention: q_out[t] = q[t, :nq] / rms * wq (plain weight); the cache row of (slot[t], pos[t]) <-
  * [k[t, :nk] / rms * wk | v[t, :nv]]. q_group / k_group 0: one norm over all nq (nk) columns at once, weight [nq] ([nk]); > 0: one norm
  * per that many consecutive columns (a head, or one score map of a head) with a weight of that size shared by the groups.
- * Pool [pages][page_size][nk + nv] and q_out of dtype dt. */
+ * cs != NULL: behind the norm the first rot_dims dimensions of every `head` columns of q and k are rotated by cs[pos[t]] (fp32
+ * [n_pos][rot_dims / 2][2]: cos, sin), dimension i paired with i + rot_dims / 2 (rot_halves) or 2i with 2i + 1. v may be k: values
+ * that are the keys as projected. Pool [pages][page_size][nk + nv] and q_out of dtype dt. */
 int omc_qk_norm_kv_store(const float* q, long long ldq, int nq, int q_group, const void* wq, const float* k, long long ldk, int nk,
-                         int k_group, const void* wk, int w_dt, const float* v, long long ldv, int nv, float eps, int T,
+                         int k_group, const void* wk, int w_dt, const float* v, long long ldv, int nv, float eps,
+                         const float* cs, int head, int rot_dims, int rot_halves, int T,
                          const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size, void* pool,
                          void* q_out, long long ldqo, int dt, void* stream);
 
-/* Sliding-window attention over such a pool: row t (position p of its slot) sees the keys j <= p with p - j < window or
- * j < keep_first (the first keys of the sequence stay visible; 0: none). score = (q . k) * scale; softcap > 0: score = softcap *
+/* Sliding-window attention over such a pool: row t (position p of its slot) sees the keys j <= p with p - j < window and
+ * floor(j / chunk) = floor(p / chunk) (chunks counted from position 0 of the sequence), or j < keep_first (the first keys of the sequence stay visible; 0: none). score = (q . k) * scale; softcap > 0: score = softcap *
  * tanh(score / softcap); dist_bias != NULL (fp32 [window, H]): score += dist_bias[p - j][h] for p - j < window; softmax;
  * out = sum_j p_j v_j. Query head h reads key/value head h / (H / G). maps >= 1 score maps per head: q is [T, H, maps, d], a cache
  * row [G, maps, d keys | G, dv values], out [T, H, maps, dv] - every map is a softmax of its own over the same values.
  * sink (fp32 [H] or NULL): the softmax denominator of head h holds one more term exp(sink[h]) - no key, no value, neither scaled
- * nor capped. gate (fp32 [T, ldg] laid out like out, or NULL): out *= act(gate), gate_act 0: as is, 1: silu, 2: sigmoid.
+ * nor capped. gate (fp32 [T, ldg] laid out like out - with gate_heads one number per head and map, [T, H, maps] - or
+ * NULL): out *= act(gate), gate_act 0: as is, 1: silu, 2: sigmoid.
  * q and pool of dtype dt, out of out_dt. dv <= 256. */
 int omc_window_attn(const void* q, long long ldq, int T, int H, int G, int d, int dv, int maps, const void* pool, int dt,
                     const int32_t* block_table, int max_pages, int page_size, const int32_t* pos, const int32_t* slot, int window,
-                    int keep_first, float scale, float softcap, const float* dist_bias, const float* sink, const float* gate,
-                    long long ldg, int gate_act, void* out, int out_dt, long long ldo, void* stream);
+                    int chunk, int keep_first, float scale, float softcap, const float* dist_bias, const float* sink, const float* gate,
+                    long long ldg, int gate_act, int gate_heads, void* out, int out_dt, long long ldo, void* stream);
 
 /* Rows of a step for an attention whose positions enter the queries and keys: per head the first rot_dims dimensions of q and k
  * are rotated pairwise, (u, v) at (2i, 2i + 1) -> (u cos a - v sin a, v cos a + u sin a) with a = position * freq[i] formed in fp32
@@ -289,15 +306,15 @@ int omc_pos_qkv_store(const float* q, long long ldq, int H, const float* k, long
                       const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size, void* pool,
                       void* q_out, long long ldqo, int dt, void* stream);
 
-/* Tensor-core version of omc_window_attn (bf16 q and pool; d and dv multiples of 16, d <= 256, dv <= 128, H / G a divisor of 64 -
- * omc_window_attn_mma_ok says 1). items: int32 [n_items][4] (first_row, n_tok, slot, first_pos), n_tok <= 64 / (H / G) consecutive
+/* Tensor-core version of omc_window_attn (bf16 q and pool; d and dv multiples of 16, d <= 256, dv <= 128, H / G <= 64 -
+ * omc_window_attn_mma_ok says 1). items: int32 [n_items][4] (first_row, n_tok, slot, first_pos), n_tok <= floor(64 / (H / G)) consecutive
  * rows of one request; items NULL: every one of the T rows is an item of its own, taken from pos / slot on the device. Same
  * results as omc_window_attn up to the bf16 rounding of the probabilities and the hardware exponentials. */
 int omc_window_attn_mma_ok(int H, int G, int d, int dv);
 int omc_window_attn_mma(const void* q, long long ldq, int T, int H, int G, int d, int dv, int maps, const void* pool,
                         const int32_t* block_table, int max_pages, int page_size, const int32_t* items, int n_items, const int32_t* pos,
-                        const int32_t* slot, int window, int keep_first, float scale, float softcap, const float* dist_bias,
-                        const float* sink, const float* gate, long long ldg, int gate_act, void* out, int out_dt, long long ldo, void* stream);
+                        const int32_t* slot, int window, int chunk, int keep_first, float scale, float softcap, const float* dist_bias,
+                        const float* sink, const float* gate, long long ldg, int gate_act, int gate_heads, void* out, int out_dt, long long ldo, void* stream);
 
 /* Differential heads: a fp32 [T, H, 2, dv] (two score maps per head) -> o = a1 - lambda * a2; o / sqrt(mean(o^2) + eps) over the
  * head's dv values; times mult; times act(gate[t, h * dv + c]) (gate fp32 or NULL; gate_act 0: as is, 1: silu, 2: sigmoid)
@@ -328,6 +345,22 @@ int omc_map_rows(float* x, long long ldx, int rows, int cols, int op, const floa
 int omc_ln_residual(const float* x, long long ldx, float alpha, const float* y, long long ldy, const float* ys, long long ldys,
                     const int32_t* slot_of, const float* w, int top, const void* nw, const void* nb, int w_dt, float eps, float* x_out,
                     long long ldxo, void* xb, int xb_dt, long long ldxb, int rows, int C, void* stream);
+
+/* Residual sum + RMS norm of the next sublayer's input (a norm in front of the sublayers), the experts' combine included:
+ *   v = x[t] + y[t] + sum_{j < top} w[t, j] * ys[slot_of[t, j]]     (y / ys NULL: no such term; slot_of < 0: skipped)
+ * -> x_out[t] = v (fp32, may be x; NULL to skip) and xb[t] = v / sqrt(mean(v^2) + eps) * nw (of xb_dt; NULL to skip). nw [C] of w_dt. */
+int omc_rms_residual(const float* x, long long ldx, const float* y, long long ldy, const float* ys, long long ldys, const int32_t* slot_of,
+                     const float* w, int top, const void* nw, int w_dt, float eps, float* x_out, long long ldxo, void* xb, int xb_dt,
+                     long long ldxb, int rows, int C, void* stream);
+
+/* h32[t, :] = table[ids[t], :] + bigram[b, :] with b = (p * mul_prev + ids[t] * mul_cur) mod buckets, p the sequence's token before row t
+ * (the row before of the same request, else prev[slot[t]]), and b = buckets for a row at position 0: bigram has buckets + 1 rows.
+ * prev (int32 [slots]) is left with the last token of every request of the step. xb[t, :] = h32[t, :] / sqrt(mean(h32^2) + eps) * nw (of
+ * xb_dt; NULL to skip). table, bigram and nw of t_dt; ids outside [0, vocab) contribute no row of the first table. single_rows as in
+ * omc_causal_conv_silu. */
+int omc_embed_bigram(const int32_t* ids, const int32_t* pos, const int32_t* slot, int T, const void* table, int t_dt, int C, int vocab,
+                     const void* bigram, int buckets, int mul_prev, int mul_cur, int32_t* prev, const void* nw, float eps, float* h32,
+                     long long ldh, void* xb, int xb_dt, long long ldxb, int single_rows, void* stream);
 
 /* Real-gated linear recurrent unit. Per channel c of `width` one fp32 state (state[slot][width]), two gates from block-diagonal
  * products whose raw outputs sit in g [T, 2 * width]: block b of `blocks` holds its n = width / blocks recurrence gates at columns

@@ -145,10 +145,12 @@ class OmChatQwen2MoeConfig(OmChatQwen2Config):
 class RotarySpec:
     """Pairwise-interleaved rotary embedding on the first `dims` dimensions of a vector: pair i = (2i, 2i + 1) turns by
     position * f_i, f_i = base^(-2i/dims). `scaling` (factor, original, fast, slow) blends f_i towards f_i / factor over a
-    linear ramp in i and multiplies cos and sin by 0.1 ln(factor) + 1 (the constants 0.1 and 0.001 are fixed by the design)."""
+    linear ramp in i and multiplies cos and sin by 0.1 ln(factor) + 1 (the constants 0.1 and 0.001 are fixed by the design).
+    halves: pair i is (i, i + dims / 2) instead."""
     dims: int
     base: float
     scaling: Optional[dict] = None
+    halves: bool = False
 
     def frequencies(self):
         """(f [dims / 2] as Python floats, multiplier of cos / sin) in double precision."""
@@ -177,8 +179,8 @@ class LatentAttentionSpec:
     """Attention whose keys and values are up-projections of a cached latent of width kv_rank plus one rotated key part of
     width rot_dim shared by the heads. q_rank: queries go through a normed latent of that width (None: one projection).
     sink: the softmax denominator has one more learned term per head. window: keys a row sees behind itself, itself included
-    (None: all). head_gate: every head's output is multiplied by a sigmoid of a projection of the mixer's input. kv_from: the
-    layer whose cached rows this one attends to (it projects no keys or values of its own and caches nothing)."""
+    (None: all). head_gate: every head's output is multiplied by a sigmoid of a projection of the mixer's input; out_gate: every
+    element of the concatenated heads is. kv_from: the layer whose cached rows this one attends to (it projects no keys or values of its own and caches nothing)."""
     heads: int
     dim: int        # unrotated query / key dimensions per head
     rot_dim: int    # rotated query / key dimensions per head
@@ -191,6 +193,7 @@ class LatentAttentionSpec:
     window: Optional[int] = None
     head_gate: bool = False
     kv_from: Optional[int] = None
+    out_gate: bool = False
 
 
 @dataclass
@@ -343,8 +346,9 @@ class ParallelMixerSpec:
 
 @dataclass
 class DenseMlpSpec:
-    """act(W_gate x + b) * (W_up x + b) -> W_down + b, act = tanh-form gelu."""
+    """act(W_gate x + b) * (W_up x + b) -> W_down + b, act = tanh-form gelu (bias False: no b)."""
     ff: int
+    bias: bool = True
 
 
 @dataclass
@@ -855,3 +859,165 @@ class MunevikConfig:
         return {"architecture": "Munevik", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps},
                 "postln_alpha": self.postln_alpha, "layers": out, "kv_page_size": self.kv_page_size, "eos_token_id": self.eos_token_id,
                 "pad_token_id": self.pad_token_id}
+
+
+# --------------------------------------------------------------------------------------------------------------------- Sorupel
+@dataclass
+class ChunkAttentionSpec:
+    """Softmax attention with grouped heads over chunks of `chunk` positions counted from the start of the sequence (None: over
+    everything earlier): a row sees the earlier rows of its own chunk. Queries and keys are RMS-normed over their whole projection, then
+    rotated; the values are the keys as projected (so a value is as wide as a key). Scores are scaled and soft-capped (0: off), the
+    denominator holds an additional 1, and every head's output is multiplied by a sigmoid of a projection of the mixer's input."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    rot: RotarySpec
+    chunk: Optional[int] = None
+    softcap: float = 0.0
+
+
+@dataclass
+class StateSpaceSpec:
+    """State-space mixer with one step size per head (Mamba-2): `heads` heads of vdim channels with a fp32 state [state, vdim] each, input
+    and output vectors B, C [state] shared by the heads of a group, a causal convolution of `conv` taps (with bias) and silu in front;
+    S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x, gated by silu(z), then RMS-normed in norm_groups equal parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int = 1
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass
+class BigramSpec:
+    """A second embedding row per token, chosen by (previous * mul_prev + current * mul_cur) mod buckets; a sequence's first token has a
+    row of its own behind the buckets."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass
+class SorupelLayerSpec:
+    type: str                      # 'latent_attention' | 'mamba2' | 'attention'
+    mixer: object                  # LatentAttentionSpec | StateSpaceSpec | ChunkAttentionSpec
+    mlp: Optional[DenseMlpSpec]
+
+
+@dataclass
+class SorupelConfig:
+    model_type: str = "sorupel"
+    vocab_size: int = 0
+    hidden_size: int = 0
+    norm_eps: float = 1e-6
+    bigram: Optional[BigramSpec] = None
+    layers: List[SorupelLayerSpec] = field(default_factory=list)
+    kv_page_size: int = 64         # engine knob: tokens per cache page
+    eos_token_id: int = -1
+    pad_token_id: int = 0
+
+    MIXERS = ("latent_attention", "mamba2", "attention")
+
+    @staticmethod
+    def _rotary(m: dict, dims: int, i: int) -> RotarySpec:
+        rot = m.get("rot") or {}
+        spec = RotarySpec(dims=int(rot.get("dims", dims)), base=float(rot.get("base", 10000.0)), halves=True)
+        if spec.dims % 2 or not 0 <= spec.dims <= dims or not spec.base > 0:
+            raise ValueError(f"layer {i}: rot.dims must be even and at most {dims}")
+        return spec
+
+    @classmethod
+    def _latent(cls, m: dict, i: int, layers: list) -> LatentAttentionSpec:
+        src = m.get("kv_from")
+        spec = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                                   scale=float(m["scale"]), rot=cls._rotary(m, int(m["rot_dim"]), i), sink=True, out_gate=True,
+                                   kv_from=int(src) if src is not None else None)
+        if min(spec.heads, spec.dim, spec.vdim, spec.kv_rank) < 1 or spec.rot_dim < 0:
+            raise ValueError(f"layer {i}: inconsistent attention sizes")
+        if spec.kv_from is not None:
+            s = layers[spec.kv_from].mixer if 0 <= spec.kv_from < i else None
+            if not isinstance(s, LatentAttentionSpec) or s.kv_from is not None:
+                raise ValueError(f"layer {i}: kv_from must name an earlier latent-attention layer with a cache of its own")
+            if (s.kv_rank, s.rot_dim, s.rot) != (spec.kv_rank, spec.rot_dim, spec.rot):
+                raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation must be those of layer {spec.kv_from}")
+        return spec
+
+    @classmethod
+    def _attention(cls, m: dict, i: int) -> ChunkAttentionSpec:
+        size = (m.get("mask") or {}).get("size")
+        spec = ChunkAttentionSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]), scale=float(m["scale"]),
+                                  rot=cls._rotary(m, int(m["dim"]), i), chunk=int(size) if size is not None else None,
+                                  softcap=float(m.get("softcap") or 0.0))
+        if min(spec.heads, spec.kv_heads, spec.dim) < 1 or spec.heads % spec.kv_heads or (spec.chunk is not None and spec.chunk < 1) or spec.softcap < 0:
+            raise ValueError(f"layer {i}: inconsistent attention sizes")
+        if int(m.get("vdim", spec.dim)) != spec.dim:
+            raise ValueError(f"layer {i}: the values are the keys, so vdim must equal dim")
+        return spec
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "SorupelConfig":
+        layers = []
+        for i, ld in enumerate(d["layers"]):
+            typ, m = ld["type"], ld["mixer"]
+            if typ == "latent_attention":
+                mix = cls._latent(m, i, layers)
+            elif typ == "attention":
+                mix = cls._attention(m, i)
+            elif typ == "mamba2":
+                mix = StateSpaceSpec(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]), groups=int(m["groups"]), conv=int(m["conv"]),
+                                     norm_groups=int(m.get("norm_groups", 1)))
+                if min(mix.heads, mix.vdim, mix.state, mix.groups, mix.conv, mix.norm_groups) < 1 or mix.heads % mix.groups or mix.inner % mix.norm_groups:
+                    raise ValueError(f"layer {i}: inconsistent state-space sizes")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {typ!r}")
+            md, mlp = ld.get("mlp"), None
+            if md:
+                if md.get("kind", "dense") != "dense":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {md.get('kind')!r}")
+                mlp = DenseMlpSpec(ff=int(md["ff"]), bias=False)
+                if mlp.ff < 1:
+                    raise ValueError(f"layer {i}: a feed-forward needs a width")
+            layers.append(SorupelLayerSpec(type=typ, mixer=mix, mlp=mlp))
+        b = (d.get("embedding") or {}).get("bigram")
+        bigram = BigramSpec(buckets=int(b["buckets"]), mul_prev=int(b["mul_prev"]), mul_cur=int(b["mul_cur"])) if b else None
+        if bigram is not None and bigram.buckets < 1:
+            raise ValueError("embedding.bigram needs at least one bucket")
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), bigram=bigram,
+                   layers=layers, kv_page_size=int(d.get("kv_page_size", 64)), eos_token_id=int(d.get("eos_token_id", -1)),
+                   pad_token_id=int(d.get("pad_token_id", 0)))
+
+    def to_dict(self) -> dict:
+        """The config.json form (round-trips through from_dict)."""
+        out = []
+        for l in self.layers:
+            m = l.mixer
+            if isinstance(m, StateSpaceSpec):
+                md = {"conv": m.conv, "groups": m.groups, "heads": m.heads, "norm_groups": m.norm_groups, "state": m.state, "vdim": m.vdim}
+            else:
+                md = {"dim": m.dim, "heads": m.heads, "rot": {"base": m.rot.base, "dims": m.rot.dims}, "scale": m.scale}
+                if isinstance(m, LatentAttentionSpec):
+                    md.update(kv_rank=m.kv_rank, rot_dim=m.rot_dim, vdim=m.vdim)
+                    if m.kv_from is not None:
+                        md["kv_from"] = m.kv_from
+                else:
+                    md.update(kv_heads=m.kv_heads, vdim=m.dim)
+                    if m.chunk is not None:
+                        md["mask"] = {"size": m.chunk}
+                    if m.softcap:
+                        md["softcap"] = m.softcap
+            out.append({"type": l.type, "mixer": md, "mlp": {"ff": l.mlp.ff, "kind": "dense"} if l.mlp is not None else None})
+        emb = {}
+        if self.bigram is not None:
+            emb["bigram"] = {"buckets": self.bigram.buckets, "mul_cur": self.bigram.mul_cur, "mul_prev": self.bigram.mul_prev}
+        return {"architecture": "Sorupel", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps}, "embedding": emb,
+                "layers": out, "kv_page_size": self.kv_page_size, "eos_token_id": self.eos_token_id, "pad_token_id": self.pad_token_id}

@@ -8,6 +8,7 @@
 //   omc_latent_kv_store  one CTA per new row: RMS norm of the latent, pairwise-interleaved rotation of the key part, append to the
 //                        row's page (fused norm + rotation + cache write)
 //   omc_rotary_q         the rotated query parts, written behind the absorbed part of each head
+//   omc_latent_rope_store  both of these in one launch, the pairs of a rotation being (2i, 2i + 1) or (i, i + dims / 2)
 //   omc_latent_attn      plain kernel, any sizes, fp32 arithmetic: one CTA per (row, head), one warp per key, online softmax with
 //                        an optional sink term exp(sink_h) that only enlarges the denominator
 // Rows of a step are addressed by (slot, position): a row sees cache entries 0..position of its slot, whether they were written
@@ -70,7 +71,7 @@ __global__ void __launch_bounds__(128) rotary_q_kernel(const TI* __restrict__ q3
 template <typename T, typename TQ>
 __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __restrict__ dkv, long long ld, int r, int dr,
                                                                 const T* __restrict__ w, float eps, const float* __restrict__ cs,
-                                                                int rot_dims, const int32_t* __restrict__ pos,
+                                                                int rot_dims, int halves, const int32_t* __restrict__ pos,
                                                                 const int32_t* __restrict__ slot,
                                                                 const int32_t* __restrict__ block_table, int max_pages, int page_size,
                                                                 T* __restrict__ pool, const TQ* __restrict__ q, long long ldq, int H, int dn,
@@ -80,6 +81,7 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
   const int p = pos[t];
   const int half = rot_dims >> 1;
   const float* csr = cs + (long long)p * rot_dims;
+  const int first = halves ? 1 : 2, apart = halves ? half : 1;   // pair i: dimensions i * first and i * first + apart
   if (dkv != nullptr && blockIdx.y == 0) {
     const float* row = dkv + (long long)t * ld;
     const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
@@ -90,9 +92,10 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
     const float rstd = 1.f / sqrtf(ss / (float)r + eps);
     for (int c = threadIdx.x; c < r; c += blockDim.x) stf(dst + c, row[c] * rstd * ldf(w + c));
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-      const float u = row[r + 2 * i], v = row[r + 2 * i + 1], co = csr[2 * i], si = csr[2 * i + 1];
-      stf(dst + r + 2 * i, u * co - v * si);
-      stf(dst + r + 2 * i + 1, v * co + u * si);
+      const int a = r + i * first, b = a + apart;
+      const float u = row[a], v = row[b], co = csr[2 * i], si = csr[2 * i + 1];
+      stf(dst + a, u * co - v * si);
+      stf(dst + b, v * co + u * si);
     }
     for (int c = rot_dims + threadIdx.x; c < dr; c += blockDim.x) stf(dst + r + c, row[r + c]);
   }
@@ -102,9 +105,10 @@ __global__ void __launch_bounds__(128) latent_rope_store_kernel(const float* __r
     const int h = h0 + i / half, j = i % half;
     const TQ* src = q + (long long)t * ldq + (long long)h * (dn + dr) + dn;
     T* qd = qcat + ((long long)t * H + h) * (r + dr) + r;
-    const float u = ldf(src + 2 * j), v = ldf(src + 2 * j + 1), co = csr[2 * j], si = csr[2 * j + 1];
-    stf(qd + 2 * j, u * co - v * si);
-    stf(qd + 2 * j + 1, v * co + u * si);
+    const int a = j * first, b = a + apart;
+    const float u = ldf(src + a), v = ldf(src + b), co = csr[2 * j], si = csr[2 * j + 1];
+    stf(qd + a, u * co - v * si);
+    stf(qd + b, v * co + u * si);
   }
   const int rest = dr - rot_dims;
   for (int i = threadIdx.x; i < nh * rest; i += blockDim.x) {
@@ -221,8 +225,8 @@ extern "C" int omc_latent_kv_store(const float* dkv, long long ld, int T, int r,
 }
 
 extern "C" int omc_latent_rope_store(const float* dkv, long long ld, int T, int r, int dr, const void* w, float eps, const float* cs,
-                                     int rot_dims, const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages,
-                                     int page_size, void* pool, const void* q, int q_dt, long long ldq, int H, int dn, void* qcat, void* qn,
+                                     int rot_dims, int rot_halves, const int32_t* pos, const int32_t* slot, const int32_t* block_table,
+                                     int max_pages, int page_size, void* pool, const void* q, int q_dt, long long ldq, int H, int dn, void* qcat, void* qn,
                                      int dt, void* stream) {
   if (cs == nullptr || pos == nullptr || q == nullptr || qcat == nullptr || T < 0 || r <= 0 || dr < 0 || rot_dims < 0 || rot_dims > dr ||
       (rot_dims & 1) || H <= 0 || dn < 0 ||
@@ -231,7 +235,7 @@ extern "C" int omc_latent_rope_store(const float* dkv, long long ld, int T, int 
   if (T == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   OMC_DT_SWITCH(dt, TT, OMC_DT_SWITCH(q_dt, TQ, {
-    latent_rope_store_kernel<TT, TQ><<<dim3(T, T <= 64 ? (H + 3) / 4 : 1), 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, pos, slot, block_table,
+    latent_rope_store_kernel<TT, TQ><<<dim3(T, T <= 64 ? (H + 3) / 4 : 1), 128, 0, st>>>(dkv, ld, r, dr, static_cast<const TT*>(w), eps, cs, rot_dims, rot_halves, pos, slot, block_table,
                                                         max_pages, page_size, static_cast<TT*>(pool), static_cast<const TQ*>(q), ldq, H, dn,
                                                         static_cast<TT*>(qcat), static_cast<TT*>(qn));
   }))

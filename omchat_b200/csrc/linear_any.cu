@@ -23,6 +23,9 @@ struct LinearArgs {
   int act;
   const void* bias;  // [N] of the weights' dtype, added before the activation (NULL: none); batch item b reads bias + b * sbias
   long long sbias;
+  const void* gate;  // [M, .] of gate_dt: outputs are multiplied by sigmoid(gate[m * ldg + b * sg + n]) (NULL: none)
+  int gate_dt;
+  long long ldg, sg;
 };
 
 __device__ __forceinline__ float apply_act(float z, int act) {
@@ -33,6 +36,13 @@ __device__ __forceinline__ float apply_act(float z, int act) {
   if (act == OMC_ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   if (act == OMC_ACT_GELU_ERF) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
   return z;
+}
+
+__device__ __forceinline__ float gate_out(float y, const LinearArgs& a, int m, int n) {
+  if (a.gate == nullptr) return y;
+  const long long at = (long long)m * a.ldg + (long long)blockIdx.z * a.sg + n;
+  const float z = a.gate_dt == OMC_DT_F32 ? static_cast<const float*>(a.gate)[at] : ldf(static_cast<const bf16_t*>(a.gate) + at);
+  return y / (1.f + expf(-z));
 }
 
 template <typename TX, typename TW, typename TY>
@@ -80,7 +90,9 @@ __global__ void __launch_bounds__(256) linear_tile_kernel(LinearArgs a) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < a.N) stf(Y + (long long)m * a.ldy + n, apply_act(acc[i][j] * a.alpha + (a.bias != nullptr ? ldf(static_cast<const TW*>(a.bias) + blockIdx.z * a.sbias + n) : 0.f), a.act));
+      if (n < a.N)
+        stf(Y + (long long)m * a.ldy + n,
+            gate_out(apply_act(acc[i][j] * a.alpha + (a.bias != nullptr ? ldf(static_cast<const TW*>(a.bias) + blockIdx.z * a.sbias + n) : 0.f), a.act), a, m, n));
     }
   }
 }
@@ -164,7 +176,7 @@ __global__ void __launch_bounds__(256, 2) linear_narrow_kernel(LinearArgs a) {
     }
     if (lane < nr) {
       const float b = a.bias != nullptr ? ldf(static_cast<const TW*>(a.bias) + blockIdx.z * a.sbias + n) : 0.f;
-      stf(Y + (long long)(m0 + lane) * a.ldy + n, apply_act(mine * a.alpha + b, a.act));
+      stf(Y + (long long)(m0 + lane) * a.ldy + n, gate_out(apply_act(mine * a.alpha + b, a.act), a, m0 + lane, n));
     }
   }
 }
@@ -256,7 +268,8 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
         if (m >= a.M || n >= a.N) continue;
         const bf16_t* bias = a.bias != nullptr ? static_cast<const bf16_t*>(a.bias) + blockIdx.z * a.sbias : nullptr;
         const float b0 = bias != nullptr ? ldf(bias + n) : 0.f, b1 = (bias != nullptr && n + 1 < a.N) ? ldf(bias + n + 1) : 0.f;
-        const float v0 = apply_act(acc[mm][nn][2 * hh] * a.alpha + b0, a.act), v1 = apply_act(acc[mm][nn][2 * hh + 1] * a.alpha + b1, a.act);
+        const float v0 = gate_out(apply_act(acc[mm][nn][2 * hh] * a.alpha + b0, a.act), a, m, n);
+        const float v1 = n + 1 < a.N ? gate_out(apply_act(acc[mm][nn][2 * hh + 1] * a.alpha + b1, a.act), a, m, n + 1) : 0.f;
         TY* dst = Y + (long long)m * a.ldy + n;
         if (pair_ok && n + 1 < a.N) {
           store_pair(dst, v0, v1);
@@ -312,10 +325,10 @@ static int launch_linear(const LinearArgs& a, int y_dt, int batch, cudaStream_t 
 
 }  // namespace omc
 
-extern "C" int omc_linear_bias(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw,
-                               long long sw, void* Y, int y_dt, long long ldy, long long sy, int M, int N, int K, int batch,
-                               float alpha, int act, const int32_t* tile_group, long long group_stride, const void* bias,
-                               long long sbias, void* stream) {
+static int run_linear(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw, long long sw, void* Y, int y_dt,
+                      long long ldy, long long sy, int M, int N, int K, int batch, float alpha, int act, const int32_t* tile_group,
+                      long long group_stride, const void* bias, long long sbias, const void* gate, int gate_dt, long long ldg, long long sg,
+                      void* stream) {
   using namespace omc;
   if (X == nullptr || W == nullptr || Y == nullptr || N <= 0 || K <= 0 || M < 0 || batch <= 0)
     return set_error(OMC_ERR_ARG, "omc_linear: bad argument");
@@ -324,7 +337,7 @@ extern "C" int omc_linear_bias(const void* X, int x_dt, long long ldx, long long
   if ((long long)((M + kLinBM - 1) / kLinBM) > 65535 || batch > 65535)
     return set_error(OMC_ERR_SHAPE, "omc_linear: more than 65535 row tiles or batch items");
   if (bias != nullptr && tile_group != nullptr) return set_error(OMC_ERR_ARG, "omc_linear: a bias excludes a tile table");
-  LinearArgs a{X, W, Y, ldx, sx, ldw, sw, ldy, sy, group_stride, tile_group, M, N, K, alpha, act, bias, sbias};
+  LinearArgs a{X, W, Y, ldx, sx, ldw, sw, ldy, sy, group_stride, tile_group, M, N, K, alpha, act, bias, sbias, gate, gate_dt, ldg, sg};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (x_dt == OMC_DT_F32 && w_dt == OMC_DT_F32) return launch_linear<float, float>(a, y_dt, batch, st);
   if (x_dt == OMC_DT_F32 && w_dt == OMC_DT_BF16) return launch_linear<float, bf16_t>(a, y_dt, batch, st);
@@ -337,9 +350,25 @@ extern "C" int omc_linear_bias(const void* X, int x_dt, long long ldx, long long
   return set_error(OMC_ERR_ARG, "omc_linear: operand dtypes must be (f32, f32), (f32, bf16) or (bf16, bf16)");
 }
 
+extern "C" int omc_linear_bias(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw,
+                               long long sw, void* Y, int y_dt, long long ldy, long long sy, int M, int N, int K, int batch,
+                               float alpha, int act, const int32_t* tile_group, long long group_stride, const void* bias,
+                               long long sbias, void* stream) {
+  return run_linear(X, x_dt, ldx, sx, W, w_dt, ldw, sw, Y, y_dt, ldy, sy, M, N, K, batch, alpha, act, tile_group, group_stride, bias, sbias, nullptr,
+                    OMC_DT_F32, 0, 0, stream);
+}
+
+extern "C" int omc_linear_gate(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw, long long sw, void* Y,
+                               int y_dt, long long ldy, long long sy, int M, int N, int K, int batch, float alpha, int act, const void* gate,
+                               int gate_dt, long long ldg, long long sg, void* stream) {
+  if (gate == nullptr || (gate_dt != OMC_DT_F32 && gate_dt != OMC_DT_BF16)) return omc::set_error(OMC_ERR_ARG, "omc_linear_gate: bad gate");
+  return run_linear(X, x_dt, ldx, sx, W, w_dt, ldw, sw, Y, y_dt, ldy, sy, M, N, K, batch, alpha, act, nullptr, 0, nullptr, 0, gate, gate_dt, ldg, sg,
+                    stream);
+}
+
 extern "C" int omc_linear(const void* X, int x_dt, long long ldx, long long sx, const void* W, int w_dt, long long ldw,
                           long long sw, void* Y, int y_dt, long long ldy, long long sy, int M, int N, int K, int batch,
                           float alpha, int act, const int32_t* tile_group, long long group_stride, void* stream) {
-  return omc_linear_bias(X, x_dt, ldx, sx, W, w_dt, ldw, sw, Y, y_dt, ldy, sy, M, N, K, batch, alpha, act, tile_group, group_stride,
-                         nullptr, 0, stream);
+  return run_linear(X, x_dt, ldx, sx, W, w_dt, ldw, sw, Y, y_dt, ldy, sy, M, N, K, batch, alpha, act, tile_group, group_stride, nullptr, 0, nullptr,
+                    OMC_DT_F32, 0, 0, stream);
 }

@@ -19,6 +19,54 @@ __global__ void __launch_bounds__(256) embed_scale_kernel(const int32_t* __restr
   }
 }
 
+// Embedding row plus a row chosen by the hashed pair (previous token, token) of the same sequence: row (prev mul_prev + cur mul_cur) mod
+// buckets of the second table, for a sequence's first token its row number `buckets` (the last one). The previous token is the row
+// before when that belongs to the same request, else the slot's state prev[slot]. The row goes to the fp32 stream, and its RMS
+// norm with weight nw, rounded, to xb (what the first sublayer reads). save_here: every row of the step is a request of its own, so
+// the slot's state is updated from here; else last_token_save_kernel does that behind this launch.
+template <typename TT, typename TB>
+__global__ void __launch_bounds__(256) embed_bigram_kernel(const int32_t* __restrict__ ids, const int32_t* __restrict__ pos,
+                                                           const int32_t* __restrict__ slot, const TT* __restrict__ table, int C, int vocab,
+                                                           const TT* __restrict__ bigram, int buckets, int mul_prev, int mul_cur,
+                                                           int32_t* __restrict__ prev, const TT* __restrict__ nw, float eps,
+                                                           float* __restrict__ h32, long long ldh, TB* __restrict__ xb, long long ldxb, int save_here) {
+  extern __shared__ float row[];  // [C]
+  __shared__ float red[33];
+  __shared__ int s_row;
+  const int t = blockIdx.x, id = ids[t];
+  if (threadIdx.x == 0) {
+    const int s = slot[t];
+    long long b = buckets;
+    if (pos[t] > 0) {
+      const long long before = (t > 0 && slot[t - 1] == s) ? ids[t - 1] : prev[s];
+      b = (before * mul_prev + (long long)id * mul_cur) % buckets;
+      if (b < 0) b += buckets;
+    }
+    s_row = (int)b;
+    if (save_here) prev[s] = id;   // read above by this thread, and by no other
+  }
+  __syncthreads();
+  const bool ok = id >= 0 && id < vocab;
+  const TT* br = bigram + (long long)s_row * C;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    const float v = (ok ? ldf(table + (long long)id * C + c) : 0.f) + ldf(br + c);
+    h32[(long long)t * ldh + c] = v;
+    row[c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (xb == nullptr) return;
+  ss = block_sum(ss, red);
+  const float rstd = 1.f / sqrtf(ss / (float)C + eps);
+  for (int c = threadIdx.x; c < C; c += blockDim.x) stf(xb + (long long)t * ldxb + c, row[c] * rstd * ldf(nw + c));   // every thread rereads only what it wrote
+}
+
+__global__ void __launch_bounds__(256) last_token_save_kernel(const int32_t* __restrict__ ids, const int32_t* __restrict__ slot, int T,
+                                                              int32_t* __restrict__ prev) {
+  const int t = blockIdx.x * blockDim.x + threadIdx.x;
+  if (t < T && (t + 1 == T || slot[t + 1] != slot[t])) prev[slot[t]] = ids[t];
+}
+
 // Embedding row plus the sinusoidal position vector: entry 2i is sin(p * f_i), entry 2i + 1 is cos(p * f_i). The angle is formed
 // and reduced in double precision (f_i arrives as a double table), so it is exact to fp32 at any position.
 template <typename TT>
@@ -199,6 +247,8 @@ __global__ void __launch_bounds__(256) tanh_cap_rows_kernel(float* __restrict__ 
 // ---- layer norm after the residual sum --------------------------------------------------------------------------------------
 //   v = alpha * x[t] + y[t] + sum_j w[t, j] * ys[slot_of[t, j]]        (y, ys: absent terms are zero)
 //   o = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * nw + nb    -> x_out[t] (fp32 stream), xb[t] (rounded: the next input)
+// RMS: the norm stands before the sublayer instead. The sum v itself is the stream (x_out[t] = v), and what the next sublayer reads is
+// xb[t] = v / sqrt(mean(v^2) + eps) * nw.
 // One CTA per row; a thread keeps its NV float4 pieces of the row in registers (the variance is taken about the mean, two block
 // reductions with one barrier each). Rows that are not laid out for float4 or too wide go through shared memory instead (VEC false).
 struct LnResArgs {
@@ -234,7 +284,7 @@ __device__ __forceinline__ float row_sum(float v, float* red) {  // red: a [NT /
   return s;
 }
 
-template <typename TW, typename TB, int NT, int NV>
+template <typename TW, typename TB, int NT, int NV, bool RMS>
 __global__ void __launch_bounds__(NT) ln_residual_kernel(LnResArgs a) {
   __shared__ float red[2][NT / 32];
   const long long t = blockIdx.x;
@@ -271,6 +321,27 @@ __global__ void __launch_bounds__(NT) ln_residual_kernel(LnResArgs a) {
     }
   }
   float s = 0.f;
+  if (RMS) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * NT + threadIdx.x) * 4;
+      if (a.x_out != nullptr && c < a.C) *reinterpret_cast<float4*>(a.x_out + t * a.ldxo + c) = v[i];
+      s = fmaf(v[i].x, v[i].x, s), s = fmaf(v[i].y, v[i].y, s), s = fmaf(v[i].z, v[i].z, s), s = fmaf(v[i].w, v[i].w, s);
+    }
+    if (a.xb == nullptr) return;
+    const float rstd = 1.f / sqrtf(row_sum<NT>(s, red[0]) / (float)a.C + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * NT + threadIdx.x) * 4;
+      if (c < a.C) {
+        float w4[4];
+        ld4(static_cast<const TW*>(a.nw) + c, w4);
+        const float o[4] = {v[i].x * rstd * w4[0], v[i].y * rstd * w4[1], v[i].z * rstd * w4[2], v[i].w * rstd * w4[3]};
+        st4(static_cast<TB*>(a.xb) + t * a.ldxb + c, o);
+      }
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < NV; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
   const float mean = row_sum<NT>(s, red[0]) / (float)a.C;
@@ -298,7 +369,7 @@ __global__ void __launch_bounds__(NT) ln_residual_kernel(LnResArgs a) {
   }
 }
 
-template <typename TW, typename TB>
+template <typename TW, typename TB, bool RMS>
 __global__ void __launch_bounds__(256) ln_residual_any_kernel(LnResArgs a) {
   extern __shared__ float row[];  // [C]
   __shared__ float red[33];
@@ -313,7 +384,14 @@ __global__ void __launch_bounds__(256) ln_residual_any_kernel(LnResArgs a) {
         if (sl >= 0) v = fmaf(a.w[t * a.top + k], a.ys[(long long)sl * a.ldys + c], v);
       }
     row[c] = v;
-    s += v;
+    s += RMS ? v * v : v;
+    if (RMS && a.x_out != nullptr) a.x_out[t * a.ldxo + c] = v;
+  }
+  if (RMS) {
+    if (a.xb == nullptr) return;
+    const float rstd = 1.f / sqrtf(block_sum(s, red) / (float)a.C + a.eps);
+    for (int c = threadIdx.x; c < a.C; c += blockDim.x) stf(static_cast<TB*>(a.xb) + t * a.ldxb + c, row[c] * rstd * ldf(static_cast<const TW*>(a.nw) + c));
+    return;
   }
   const float mean = block_sum(s, red) / (float)a.C;
   s = 0.f;
@@ -329,27 +407,27 @@ __global__ void __launch_bounds__(256) ln_residual_any_kernel(LnResArgs a) {
   }
 }
 
-template <typename TW, typename TB>
+template <typename TW, typename TB, bool RMS>
 static int launch_ln_residual(const LnResArgs& a, int rows, cudaStream_t st) {
   auto al = [](const void* p, size_t n) { return p == nullptr || reinterpret_cast<uintptr_t>(p) % n == 0; };
   const bool vec = a.C % 4 == 0 && a.C <= 8192 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ldys % 4 == 0 && a.ldxo % 4 == 0 && a.ldxb % 4 == 0 &&
                    al(a.x, 16) && al(a.y, 16) && al(a.ys, 16) && al(a.x_out, 16) && al(a.nw, 4 * sizeof(TW)) && al(a.nb, 4 * sizeof(TW)) &&
                    al(a.xb, 4 * sizeof(TB));
   if (vec) {
-    if (a.C <= 256) ln_residual_kernel<TW, TB, 64, 1><<<rows, 64, 0, st>>>(a);
-    else if (a.C <= 512) ln_residual_kernel<TW, TB, 128, 1><<<rows, 128, 0, st>>>(a);
-    else if (a.C <= 1024) ln_residual_kernel<TW, TB, 256, 1><<<rows, 256, 0, st>>>(a);
-    else if (a.C <= 2048) ln_residual_kernel<TW, TB, 256, 2><<<rows, 256, 0, st>>>(a);
-    else if (a.C <= 4096) ln_residual_kernel<TW, TB, 256, 4><<<rows, 256, 0, st>>>(a);
-    else ln_residual_kernel<TW, TB, 256, 8><<<rows, 256, 0, st>>>(a);
+    if (a.C <= 256) ln_residual_kernel<TW, TB, 64, 1, RMS><<<rows, 64, 0, st>>>(a);
+    else if (a.C <= 512) ln_residual_kernel<TW, TB, 128, 1, RMS><<<rows, 128, 0, st>>>(a);
+    else if (a.C <= 1024) ln_residual_kernel<TW, TB, 256, 1, RMS><<<rows, 256, 0, st>>>(a);
+    else if (a.C <= 2048) ln_residual_kernel<TW, TB, 256, 2, RMS><<<rows, 256, 0, st>>>(a);
+    else if (a.C <= 4096) ln_residual_kernel<TW, TB, 256, 4, RMS><<<rows, 256, 0, st>>>(a);
+    else ln_residual_kernel<TW, TB, 256, 8, RMS><<<rows, 256, 0, st>>>(a);
   } else {
     const size_t smem = (size_t)a.C * sizeof(float);
     if (smem > 200 * 1024) return set_error(OMC_ERR_SHAPE, "omc_ln_residual: row too wide for shared memory");
     if (smem > 48 * 1024) {
-      cudaError_t e = cudaFuncSetAttribute(ln_residual_any_kernel<TW, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaError_t e = cudaFuncSetAttribute(ln_residual_any_kernel<TW, TB, RMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return set_error(OMC_ERR_CUDA, cudaGetErrorString(e));
     }
-    ln_residual_any_kernel<TW, TB><<<rows, 256, smem, st>>>(a);
+    ln_residual_any_kernel<TW, TB, RMS><<<rows, 256, smem, st>>>(a);
   }
   return check_launch("omc_ln_residual");
 }
@@ -469,5 +547,41 @@ extern "C" int omc_ln_residual(const float* x, long long ldx, float alpha, const
   const LnResArgs a{x, ldx, alpha, y, y != nullptr ? ldy : 0, ys, ys != nullptr ? ldys : 0, slot_of, w, top, nw, nb, eps, x_out,
                     x_out != nullptr ? ldxo : 0, xb, xb != nullptr ? ldxb : 0, C};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(xb_dt, TB, { return (launch_ln_residual<TW, TB>(a, rows, st)); }))
+  OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(xb_dt, TB, { return (launch_ln_residual<TW, TB, false>(a, rows, st)); }))
+}
+
+extern "C" int omc_rms_residual(const float* x, long long ldx, const float* y, long long ldy, const float* ys, long long ldys, const int32_t* slot_of,
+                                const float* w, int top, const void* nw, int w_dt, float eps, float* x_out, long long ldxo, void* xb, int xb_dt,
+                                long long ldxb, int rows, int C, void* stream) {
+  if (x == nullptr || (xb != nullptr && nw == nullptr) || (x_out == nullptr && xb == nullptr) || rows < 0 || C <= 0 ||
+      (ys != nullptr && (slot_of == nullptr || w == nullptr || top <= 0)))
+    return set_error(OMC_ERR_ARG, "omc_rms_residual: bad argument");
+  if (rows == 0) return OMC_OK;
+  const LnResArgs a{x, ldx, 1.f, y, y != nullptr ? ldy : 0, ys, ys != nullptr ? ldys : 0, slot_of, w, top, nw, nullptr, eps, x_out,
+                    x_out != nullptr ? ldxo : 0, xb, xb != nullptr ? ldxb : 0, C};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(xb_dt, TB, { return (launch_ln_residual<TW, TB, true>(a, rows, st)); }))
+}
+
+extern "C" int omc_embed_bigram(const int32_t* ids, const int32_t* pos, const int32_t* slot, int T, const void* table, int t_dt, int C, int vocab,
+                                const void* bigram, int buckets, int mul_prev, int mul_cur, int32_t* prev, const void* nw, float eps, float* h32,
+                                long long ldh, void* xb, int xb_dt, long long ldxb, int single_rows, void* stream) {
+  if (ids == nullptr || pos == nullptr || slot == nullptr || table == nullptr || bigram == nullptr || prev == nullptr || h32 == nullptr || T < 0 || C <= 0 ||
+      buckets <= 0 || mul_prev < 0 || mul_cur < 0 || (xb != nullptr && nw == nullptr))
+    return set_error(OMC_ERR_ARG, "omc_embed_bigram: bad argument");
+  if (T == 0) return OMC_OK;
+  const size_t smem = (size_t)C * sizeof(float);
+  if (smem > 200 * 1024) return set_error(OMC_ERR_SHAPE, "omc_embed_bigram: row too wide for shared memory");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  OMC_DT_SWITCH(t_dt, TT, OMC_DT_SWITCH(xb_dt, TB, {
+    if (smem > 48 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(embed_bigram_kernel<TT, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return set_error(OMC_ERR_CUDA, cudaGetErrorString(e));
+    }
+    embed_bigram_kernel<TT, TB><<<T, 256, smem, st>>>(ids, pos, slot, static_cast<const TT*>(table), C, vocab, static_cast<const TT*>(bigram), buckets,
+                                                      mul_prev, mul_cur, prev, static_cast<const TT*>(nw), eps, h32, ldh, static_cast<TB*>(xb), ldxb,
+                                                      single_rows);
+  }))
+  if (!single_rows) last_token_save_kernel<<<(T + 255) / 256, 256, 0, st>>>(ids, slot, T, prev);
+  return check_launch("omc_embed_bigram");
 }

@@ -1,7 +1,8 @@
 // Mixers that carry a fixed-size state per sequence instead of a growing cache: a short causal convolution per channel whose
 // last inputs are state, and the family of linear-state recurrences
-//     S <- diag(g_t) S;   u_t = beta_t (v_t - S^T k_t)  (delta rule)  or  u_t = v_t  (plain outer-product sum);
-//     S <- S + k_t u_t^T;   o_t = S^T q_t
+//     S <- diag(g_t) S;   u_t = beta_t (v_t - S^T k_t)  (delta rule)  or  u_t = v_t  (plain outer-product sum)
+//                         or  u_t = dt_t v_t with g_t = exp(-A dt_t)  (state-space form: one step size per token and head);
+//     S <- S + k_t u_t^T;   o_t = S^T q_t  (state-space form: + D v_t)
 // with the decay g_t constant per head, one per token and head, or one per token, head and key channel, and the gated RMS norm
 // that follows them. Rows of a step are addressed by (slot, position); the rows of one request are consecutive and ascending.
 // A portion that starts at position 0 starts from a zero state, so a slot needs no clearing when it is handed to a new request.
@@ -252,14 +253,16 @@ struct ScanArgs {
   int silu_in;         // q, k, v pass silu on the way in
   int decay_mode;      // 0: decay_const[h]; 1: a[t, h]; 2: a[t, h * dim + i]  (1, 2: g = exp(-exp(A_log[h]) softplus(a + dt_bias))); 3: g = a[t, h * dim + i];
                        // 4: g = sigmoid(a[t, h * dim + i] + dt_bias[h * dim + i])^decay_pow; 5: a[t, h * dim + i] holds g - 1
-                       // (4 and 5 apply the decay as S + (g - 1) S)
+                       // (4 and 5 apply the decay as S + (g - 1) S); 6: dt = softplus(a[t, h] + dt_bias[h]), g = exp(-exp(A_log[h]) dt),
+                       // u = dt v, o = S^T q + D[h] v (the decay as S + expm1(.) S)
   float decay_pow;     // mode 4
   float out_scale;     // o_t = out_scale * S^T q_t (a query scale, applied to the read-out)
   const float* decay_const;
   const float* a;
   long long lda;
   const float* A_log;    // fp32 [H]
-  const float* dt_bias;  // fp32 [H] (mode 1) or [H * dim] (mode 2)
+  const float* dt_bias;  // fp32 [H] (modes 1, 6) or [H * dim] (mode 2)
+  const float* D;        // fp32 [H] (mode 6) or NULL
   const float* beta;     // raw [T, ldb]: beta = sigmoid; NULL: no delta correction (u = v)
   long long ldb;
   float* state;          // [slots][H][dim][vdim]
@@ -304,13 +307,15 @@ __device__ __forceinline__ int scan_place(int i) { return (i / DPT) * (DPT + 4) 
 // Two stages of kScanTok tokens each: the raw inputs of the next chunk arrive by cp.async while the current chunk is computed;
 // after arrival one pass turns them in place into what the recurrence uses (silu, decays, sigmoid). VEC: 16-byte copies
 // (every row starts on a 16-byte boundary and the widths are multiples of four), else 4-byte copies.
-template <int DPT, bool VEC>
+// KIND: what enters the state - v itself, the delta rule's correction, or dt v (decay mode 6).
+enum { kScanPlain = 0, kScanDelta = 1, kScanStep = 2 };
+template <int DPT, bool VEC, int KIND>
 __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_kernel(ScanArgs a) {
   extern __shared__ __align__(16) float sm[];
   constexpr int PITCH = kScanLanes * (DPT + 4);
   const int dim = a.dim;
-  const bool chan = a.decay_mode >= 2;   // one decay per key channel: computed here (2, 4) or given (3, 5)
-  const bool minus1 = a.decay_mode >= 4;  // the staged value is the decay minus one
+  const bool chan = KIND != kScanStep && a.decay_mode >= 2;   // one decay per key channel: computed here (2, 4) or given (3, 5)
+  const bool minus1 = KIND == kScanStep || a.decay_mode >= 4;  // the staged value is the decay minus one
   const int stage_floats = kScanTok * PITCH * (chan ? 3 : 2) + kScanTok * kScanCols + 2 * kScanTok;
   const int h = blockIdx.y, kvh = h / (a.H / a.G);
   const int col0 = blockIdx.x * kScanCols;
@@ -321,15 +326,22 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
   const bool ok0 = col < a.vdim, ok1 = col + 1 < a.vdim;
   for (int e = tid; e < 2 * stage_floats; e += blockDim.x) sm[e] = 0.f;   // the pads stay zero: they meet zero state only
   float* S = a.state + (((long long)a.slot[r0] * a.H + h) * dim) * a.vdim;
+  const bool pairs = a.vdim % 2 == 0;   // columns (col, col + 1) lie on an 8-byte boundary
   f32x2 st[DPT];   // state elements (lane * DPT + r, col) and (lane * DPT + r, col + 1)
   const bool fresh = a.pos[r0] == 0;
 #pragma unroll
   for (int r = 0; r < DPT; ++r) {
     const int i = lane * DPT + r;
     const bool ld = !fresh && i < dim;
-    st[r] = pack2((ld && ok0) ? S[(long long)i * a.vdim + col] : 0.f, (ld && ok1) ? S[(long long)i * a.vdim + col + 1] : 0.f);
+    if (pairs) {   // both columns as one access
+      const float2 e = ld && ok0 ? *reinterpret_cast<const float2*>(S + (long long)i * a.vdim + col) : make_float2(0.f, 0.f);
+      st[r] = pack2(e.x, e.y);
+    } else {
+      st[r] = pack2((ld && ok0) ? S[(long long)i * a.vdim + col] : 0.f, (ld && ok1) ? S[(long long)i * a.vdim + col + 1] : 0.f);
+    }
   }
-  const float A = (a.decay_mode == 1 || a.decay_mode == 2) ? expf(a.A_log[h]) : 0.f;
+  const float A = (KIND == kScanStep || a.decay_mode == 1 || a.decay_mode == 2) ? expf(a.A_log[h]) : 0.f;
+  const float Dh = (KIND == kScanStep && a.D != nullptr) ? a.D[h] : 0.f;
   const float gconst = a.decay_mode == 0 ? a.decay_const[h] : 1.f;
   __syncthreads();
 
@@ -364,8 +376,8 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
       }
     }
     if (tid < n) {
-      if (a.beta != nullptr) cp_async4(sb + tid, a.beta + (long long)(c0 + tid) * a.ldb + h);
-      if (a.decay_mode == 1) cp_async4(sg + tid, a.a + (long long)(c0 + tid) * a.lda + h);
+      if (KIND == kScanDelta) cp_async4(sb + tid, a.beta + (long long)(c0 + tid) * a.ldb + h);
+      if (KIND == kScanStep || a.decay_mode == 1) cp_async4(sg + tid, a.a + (long long)(c0 + tid) * a.lda + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -400,8 +412,14 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
     }
     if (a.silu_in)
       for (int e = tid; e < n * kScanCols; e += blockDim.x) sv[e] = silu_f(sv[e]);
-    if (tid < n) {
-      sb[tid] = a.beta != nullptr ? sigmoid_f(sb[tid]) : 1.f;
+    if (KIND == kScanStep) {
+      if (tid < n) {
+        const float dt = softplus_f(sg[tid] + a.dt_bias[h]);
+        sb[tid] = dt;
+        sg[tid] = expm1f(-A * dt);
+      }
+    } else if (tid < n) {
+      sb[tid] = KIND == kScanDelta ? sigmoid_f(sb[tid]) : 1.f;
       if (a.decay_mode == 1) sg[tid] = expf(-A * softplus_f(sg[tid] + a.dt_bias[h]));
       else if (a.decay_mode == 0) sg[tid] = gconst;
     }
@@ -426,15 +444,21 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
             st[r] = mul2(st[r], pack2(gv.x, gv.x)), st[r + 1] = mul2(st[r + 1], pack2(gv.y, gv.y));
             st[r + 2] = mul2(st[r + 2], pack2(gv.z, gv.z)), st[r + 3] = mul2(st[r + 3], pack2(gv.w, gv.w));
           }
+        } else if (minus1) {
+          st[r] = fma2(st[r], gh, st[r]), st[r + 1] = fma2(st[r + 1], gh, st[r + 1]);
+          st[r + 2] = fma2(st[r + 2], gh, st[r + 2]), st[r + 3] = fma2(st[r + 3], gh, st[r + 3]);
         } else {
           st[r] = mul2(st[r], gh), st[r + 1] = mul2(st[r + 1], gh), st[r + 2] = mul2(st[r + 2], gh), st[r + 3] = mul2(st[r + 3], gh);
         }
-        da = fma2(st[r], k2[r], da), db = fma2(st[r + 1], k2[r + 1], db);
-        da = fma2(st[r + 2], k2[r + 2], da), db = fma2(st[r + 3], k2[r + 3], db);
+        if (KIND == kScanDelta) {
+          da = fma2(st[r], k2[r], da), db = fma2(st[r + 1], k2[r + 1], db);
+          da = fma2(st[r + 2], k2[r + 2], da), db = fma2(st[r + 3], k2[r + 3], db);
+        }
       }
       const float2 vv = *reinterpret_cast<const float2*>(sv + tt * kScanCols + 2 * cp);
       float u0 = vv.x, u1 = vv.y;
-      if (a.beta != nullptr) {
+      if (KIND == kScanStep) u0 *= sb[tt], u1 *= sb[tt];
+      if (KIND == kScanDelta) {
         float a0, a1, b0, b1;
         unpack2(da, a0, a1);
         unpack2(db, b0, b1);
@@ -469,6 +493,7 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
       }
       if (lane == 0) {
         float* dst = a.out + (long long)(c0 + tt) * a.ldo + h * a.vdim + col;
+        if (KIND == kScanStep) o0 = fmaf(Dh, vv.x, o0), o1 = fmaf(Dh, vv.y, o1);
         if (ok0) dst[0] = o0 * a.out_scale;
         if (ok1) dst[1] = o1 * a.out_scale;
       }
@@ -480,8 +505,12 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
     const int i = lane * DPT + r;
     float lo, hi;
     unpack2(st[r], lo, hi);
-    if (i < dim && ok0) S[(long long)i * a.vdim + col] = lo;
-    if (i < dim && ok1) S[(long long)i * a.vdim + col + 1] = hi;
+    if (pairs) {
+      if (i < dim && ok0) *reinterpret_cast<float2*>(S + (long long)i * a.vdim + col) = make_float2(lo, hi);
+    } else {
+      if (i < dim && ok0) S[(long long)i * a.vdim + col] = lo;
+      if (i < dim && ok1) S[(long long)i * a.vdim + col + 1] = hi;
+    }
   }
 }
 
@@ -527,6 +556,71 @@ __global__ void __launch_bounds__(256) gated_rms_kernel(const float* __restrict_
   }
 }
 
+
+// The gate in front of the norm: v = x * act(gate), y = v / sqrt(mean(v^2) + eps) * w with the mean over each of `groups` equal parts of
+// the row and a weight for every column. NT threads per (row, part); a thread keeps its elements in registers (VEC: four neighbours
+// at a time), parts too wide for that are read twice.
+constexpr int kGateRmsRegs = 8;   // elements (VEC: float4 pieces) a thread keeps
+template <typename TG, typename TW, typename TY, bool VEC>
+__global__ void __launch_bounds__(256) gate_rms_kernel(const float* __restrict__ x, long long ldx, int n, const TW* __restrict__ w, float eps,
+                                                       const TG* __restrict__ gate, long long ldg, int gate_act, TY* __restrict__ y, long long ldy) {
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  const long long c0 = (long long)blockIdx.y * n;
+  const float* xr = x + t * ldx + c0;
+  const TG* gr = gate + t * ldg + c0;
+  auto act = [&](float z) { return gate_act == 1 ? silu_f(z) : (gate_act == 2 ? sigmoid_f(z) : z); };
+  constexpr int V = VEC ? 4 : 1;
+  float keep[kGateRmsRegs][V];
+  float ss = 0.f;
+  auto value = [&](int c, float (&v)[V]) {
+    if constexpr (VEC) {
+      float g[4];
+      ld4(xr + c, v);
+      ld4(gr + c, g);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] *= act(g[i]);
+    } else {
+      v[0] = xr[c] * act(ldf(gr + c));
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < kGateRmsRegs; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < n) {
+      value(c, keep[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(keep[i][e], keep[i][e], ss);
+    }
+  }
+  for (int c = (kGateRmsRegs * blockDim.x + threadIdx.x) * V; c < n; c += blockDim.x * V) {
+    float v[V];
+    value(c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+  }
+  const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  auto put = [&](int c, const float (&v)[V]) {
+    if constexpr (VEC) {
+      float wv[4];
+      ld4(w + c0 + c, wv);
+      const float o[4] = {v[0] * rstd * wv[0], v[1] * rstd * wv[1], v[2] * rstd * wv[2], v[3] * rstd * wv[3]};
+      st4(y + t * ldy + c0 + c, o);
+    } else {
+      stf(y + t * ldy + c0 + c, v[0] * rstd * ldf(w + c0 + c));
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < kGateRmsRegs; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < n) put(c, keep[i]);
+  }
+  for (int c = (kGateRmsRegs * blockDim.x + threadIdx.x) * V; c < n; c += blockDim.x * V) {
+    float v[V];
+    value(c, v);
+    put(c, v);
+  }
+}
 
 // ---- tanh norm + input convolution of a sublayer ----------------------------------------------------------------------------
 // What a sublayer of a "tanh-norm" decoder reads: with the stream row x (optionally first updated by the previous sublayer's
@@ -1004,47 +1098,55 @@ extern "C" int omc_causal_conv_silu(const float* x, long long ldx, int T, int ch
 
 extern "C" int omc_linear_state_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
                                      int silu_in, int decay_mode, const float* decay_const, const float* a, long long lda,
-                                     const float* A_log, const float* dt_bias, const float* beta, long long ldb, float* state,
+                                     const float* A_log, const float* dt_bias, const float* D, const float* beta, long long ldb, float* state,
                                      float* out, long long ldo, const int32_t* row_begin, int portions, const int32_t* pos,
                                      const int32_t* slot, int H, int G, int dim, int vdim, float decay_pow, float out_scale, void* stream) {
   if (q == nullptr || k == nullptr || v == nullptr || state == nullptr || out == nullptr || row_begin == nullptr || pos == nullptr ||
-      slot == nullptr || portions < 0 || H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || decay_mode < 0 || decay_mode > 5 ||
-      (decay_mode == 0 && decay_const == nullptr) || (decay_mode != 0 && a == nullptr) ||
-      ((decay_mode == 1 || decay_mode == 2) && (A_log == nullptr || dt_bias == nullptr)))
+      slot == nullptr || portions < 0 || H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || decay_mode < 0 || decay_mode > 6 ||
+      (decay_mode == 0 && decay_const == nullptr) || (decay_mode != 0 && a == nullptr) || (decay_mode == 6 && beta != nullptr) || (D != nullptr && decay_mode != 6) ||
+      ((decay_mode == 1 || decay_mode == 2 || decay_mode == 6) && (A_log == nullptr || dt_bias == nullptr)))
     return set_error(OMC_ERR_ARG, "omc_linear_state_scan: bad argument");
   if (portions == 0) return OMC_OK;
   if (dim > 256) return set_error(OMC_ERR_SHAPE, "omc_linear_state_scan: key width above 256");
   if (portions > 65535 || H > 65535) return set_error(OMC_ERR_SHAPE, "omc_linear_state_scan: more than 65535 portions or heads");
-  ScanArgs s{q, k, v, ldq, ldk, ldv, silu_in, decay_mode, decay_pow, out_scale, decay_const, a, lda, A_log, dt_bias, beta, ldb, state, out, ldo,
+  ScanArgs s{q, k, v, ldq, ldk, ldv, silu_in, decay_mode, decay_pow, out_scale, decay_const, a, lda, A_log, dt_bias, D, beta, ldb, state, out, ldo,
              row_begin, pos, slot, H, G, dim, vdim};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int dpt = dim <= 32 ? 4 : (dim <= 64 ? 8 : (dim <= 128 ? 16 : 32));   // key channels per thread: dim / 8 lanes, rounded up to a float4
-  const size_t stage_floats = (size_t)kScanTok * kScanLanes * (dpt + 4) * (decay_mode >= 2 ? 3 : 2) + kScanTok * kScanCols + 2 * kScanTok;
+  const bool chan = decay_mode >= 2 && decay_mode <= 5;
+  const size_t stage_floats = (size_t)kScanTok * kScanLanes * (dpt + 4) * (chan ? 3 : 2) + kScanTok * kScanCols + 2 * kScanTok;
   const size_t smem = 2 * stage_floats * sizeof(float);
   dim3 grid((vdim + kScanCols - 1) / kScanCols, H, portions);
   const int threads = kScanCols / 2 * kScanLanes;
   auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const bool vec = dim % 4 == 0 && vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && al16(q) && al16(k) && al16(v) &&
-                   (decay_mode < 2 || (lda % 4 == 0 && al16(a)));
-#define OMC_SCAN_LAUNCH(DPT, VEC)                                                                                        \
-  do {                                                                                                                   \
-    static bool attr_done[kMaxDevices] = {};                                                                             \
-    if (!attr_done[cur_device()]) {                                                                                      \
-      cudaFuncSetAttribute(linear_state_scan_kernel<DPT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024); \
-      attr_done[cur_device()] = true;                                                                                    \
-    }                                                                                                                    \
-    linear_state_scan_kernel<DPT, VEC><<<grid, threads, smem, st>>>(s);                                                  \
+                   (!chan || (lda % 4 == 0 && al16(a)));
+#define OMC_SCAN_LAUNCH(DPT, VEC, KIND)                                                                                        \
+  do {                                                                                                                         \
+    static bool attr_done[kMaxDevices] = {};                                                                                   \
+    if (!attr_done[cur_device()]) {                                                                                            \
+      cudaFuncSetAttribute(linear_state_scan_kernel<DPT, VEC, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024); \
+      attr_done[cur_device()] = true;                                                                                          \
+    }                                                                                                                          \
+    linear_state_scan_kernel<DPT, VEC, KIND><<<grid, threads, smem, st>>>(s);                                                  \
   } while (0)
-#define OMC_SCAN_DPT(DPT)          \
-  do {                             \
-    if (vec) OMC_SCAN_LAUNCH(DPT, true); \
-    else OMC_SCAN_LAUNCH(DPT, false);    \
+#define OMC_SCAN_KIND(DPT, VEC)                                         \
+  do {                                                                  \
+    if (decay_mode == 6) OMC_SCAN_LAUNCH(DPT, VEC, kScanStep);          \
+    else if (beta != nullptr) OMC_SCAN_LAUNCH(DPT, VEC, kScanDelta);    \
+    else OMC_SCAN_LAUNCH(DPT, VEC, kScanPlain);                         \
+  } while (0)
+#define OMC_SCAN_DPT(DPT)              \
+  do {                                 \
+    if (vec) OMC_SCAN_KIND(DPT, true); \
+    else OMC_SCAN_KIND(DPT, false);    \
   } while (0)
   if (dpt == 4) OMC_SCAN_DPT(4);
   else if (dpt == 8) OMC_SCAN_DPT(8);
   else if (dpt == 16) OMC_SCAN_DPT(16);
   else OMC_SCAN_DPT(32);
 #undef OMC_SCAN_DPT
+#undef OMC_SCAN_KIND
 #undef OMC_SCAN_LAUNCH
   return check_launch("omc_linear_state_scan");
 }
@@ -1061,6 +1163,28 @@ extern "C" int omc_gated_rms_rows(const float* x, long long ldx, int rows, int g
                                                                                  gate, ldg, gate_act, static_cast<TY*>(y), ldy);
   }))
   return check_launch("omc_gated_rms_rows");
+}
+
+extern "C" int omc_gate_rms_rows(const float* x, long long ldx, int rows, int groups, int n, const void* w, int w_dt, float eps, const void* gate,
+                                 int gate_dt, long long ldg, int gate_act, void* y, int y_dt, long long ldy, void* stream) {
+  if (x == nullptr || w == nullptr || gate == nullptr || y == nullptr || rows < 0 || groups <= 0 || n <= 0 || gate_act < 0 || gate_act > 2)
+    return set_error(OMC_ERR_ARG, "omc_gate_rms_rows: bad argument");
+  if (groups > 65535) return set_error(OMC_ERR_SHAPE, "omc_gate_rms_rows: more than 65535 parts");
+  if (rows == 0) return OMC_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  auto al = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool vec = n % 4 == 0 && ldx % 4 == 0 && ldg % 4 == 0 && ldy % 4 == 0 && al(x) && al(gate) && al(y) && al(w);
+  const int per = vec ? 4 : 1;
+  int threads = 32;   // about one or two pieces per thread up to 256 threads
+  while (threads < 256 && threads * per * 2 < n) threads <<= 1;
+  const dim3 grid(rows, groups);
+  OMC_DT_SWITCH(gate_dt, TG, OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(y_dt, TY, {
+    if (vec) gate_rms_kernel<TG, TW, TY, true><<<grid, threads, 0, st>>>(x, ldx, n, static_cast<const TW*>(w), eps, static_cast<const TG*>(gate), ldg, gate_act,
+                                                                         static_cast<TY*>(y), ldy);
+    else gate_rms_kernel<TG, TW, TY, false><<<grid, threads, 0, st>>>(x, ldx, n, static_cast<const TW*>(w), eps, static_cast<const TG*>(gate), ldg, gate_act,
+                                                                      static_cast<TY*>(y), ldy);
+  })))
+  return check_launch("omc_gate_rms_rows");
 }
 
 extern "C" int omc_map_rows(float* x, long long ldx, int rows, int cols, int op, const float* A_log, const float* bias, int group,

@@ -1,16 +1,18 @@
-// Sliding-window softmax attention over a paged key/value cache, without rotation: positions enter through a bias that depends on
-// the distance between query and key only. Per cached token one row [kv_heads * dim keys | kv_heads * vdim values].
+// Sliding-window and chunked softmax attention over a paged key/value cache: positions enter through a bias that depends on the
+// distance between query and key only, or are rotated into queries and keys before the keys are cached. Per cached token one row
+// [kv_heads * dim keys | kv_heads * vdim values].
 //
 //   omc_qk_norm_kv_store: the rows of a step -> normed queries, and normed keys + values appended to the pages (one RMS norm over the
-//                         whole projection, or one per group of columns - a head, or a score map of a head - with a shared weight)
+//                         whole projection, or one per group of columns - a head, or a score map of a head - with a shared weight),
+//                         optionally rotated per head behind the norm
 //   omc_window_attn:      score = (q . k) * scale -> softcap * tanh(score / softcap) -> + dist_bias[i - j][head] -> softmax over the
-//                         keys j with 0 <= i - j < window, and the first keep_first keys of the sequence whatever their distance
-//                         -> weighted sum of values. maps > 1: every head has that many score maps (queries and keys of their own)
+//                         keys j with 0 <= i - j < window and floor(j / chunk) = floor(i / chunk), and the first keep_first keys of
+//                         the sequence whatever their distance -> weighted sum of values. maps > 1: every head has that many score maps (queries and keys of their own)
 //                         over the same values; the maps come out side by side.
 //   omc_diff_heads_gate:  two maps -> o = a1 - lambda a2, RMS norm over the head, a constant factor, an elementwise gate
 // The distance bias arrives as a table [window, heads] that the host builds (here from a bucketed learned table; any function of
 // the distance fits). Prompt portions and decoded tokens are one case: row t at position pos[t] of slot[t] reads the cached
-// entries max(0, pos - window + 1) .. pos of its slot, which the store kernel of the same step has written.
+// entries max(0, pos - window + 1, pos - pos % chunk) .. pos of its slot, which the store kernel of the same step has written.
 // The plain kernel: fp32 arithmetic, one CTA per (row, head), a warp per key, lanes across the head dimension.
 #include <math.h>
 
@@ -21,17 +23,37 @@ namespace omc {
 constexpr int kWinWarps = 4;
 constexpr int kWinMaxPerLane = 8;  // value width up to 256
 
-// One CTA per row. q: RMS norm with a plain weight -> q_out; k likewise -> page; v copied -> page. group 0: one norm over all
-// columns, weight [n]; group > 0: one norm per `group` consecutive columns (a warp each), weight [group] shared by the groups.
+// Rotation of the first `dims` dimensions of every `width` consecutive columns by a host-built table of (cos, sin) [position][dims / 2][2]
+// (cs: this row's part of it, NULL: none). halves: dimension i pairs with i + dims / 2, else the pairs are (2i, 2i + 1).
+struct HeadRotation {
+  const float* cs;
+  int width, dims, halves;
+};
+// Column c of x * w (wi: the weight's column) times rstd, turned.
+template <typename TW>
+__device__ __forceinline__ float norm_rot_value(const float* __restrict__ x, const TW* __restrict__ w, int c, int wi, float rstd, const HeadRotation& rot) {
+  const float v = x[c] * rstd * ldf(w + wi);
+  if (rot.cs == nullptr) return v;
+  const int i = c % rot.width;
+  if (i >= rot.dims) return v;
+  const int half = rot.dims >> 1;
+  const bool second = rot.halves ? i >= half : (i & 1);
+  const int f = rot.halves ? (second ? i - half : i) : i >> 1, to = rot.halves ? (second ? -half : half) : (second ? -1 : 1);
+  const float o = x[c + to] * rstd * ldf(w + wi + to), co = rot.cs[2 * f], si = rot.cs[2 * f + 1];
+  return second ? v * co + o * si : v * co - o * si;
+}
+
+// One CTA per row. q: RMS norm with a plain weight (and rotation) -> q_out; k likewise -> page; v copied -> page. group 0: one norm over
+// all columns, weight [n]; group > 0: one norm per `group` consecutive columns (a warp each), weight [group] shared by the groups.
 template <typename TW, typename TD>
 __device__ __forceinline__ void rms_to(const float* __restrict__ x, int n, int group, const TW* __restrict__ w, float eps,
-                                       TD* __restrict__ dst, float* red) {
+                                       TD* __restrict__ dst, float* red, const HeadRotation& rot) {
   if (group <= 0) {
     float ss = 0.f;
     for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
     ss = block_sum(ss, red);
     const float rstd = 1.f / sqrtf(ss / (float)n + eps);
-    for (int c = threadIdx.x; c < n; c += blockDim.x) stf(dst + c, x[c] * rstd * ldf(w + c));
+    for (int c = threadIdx.x; c < n; c += blockDim.x) stf(dst + c, norm_rot_value(x, w, c, c, rstd, rot));
     return;
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -41,7 +63,7 @@ __device__ __forceinline__ void rms_to(const float* __restrict__ x, int n, int g
     for (int c = lane; c < group; c += 32) ss = fmaf(xg[c], xg[c], ss);
     ss = seq_warp_sum(ss);
     const float rstd = 1.f / sqrtf(ss / (float)group + eps);
-    for (int c = lane; c < group; c += 32) stf(dst + g * group + c, xg[c] * rstd * ldf(w + c));
+    for (int c = lane; c < group; c += 32) stf(dst + g * group + c, norm_rot_value(xg, w, c, c, rstd, rot));
   }
 }
 
@@ -49,7 +71,7 @@ template <typename TW, typename TC>
 __global__ void __launch_bounds__(256) qk_norm_kv_store_kernel(const float* __restrict__ q, long long ldq, int nq, int q_group,
                                                                const TW* __restrict__ wq, const float* __restrict__ k, long long ldk,
                                                                int nk, int k_group, const TW* __restrict__ wk, const float* __restrict__ v,
-                                                               long long ldv, int nv, float eps, const int32_t* __restrict__ pos,
+                                                               long long ldv, int nv, float eps, HeadRotation rot, const int32_t* __restrict__ pos,
                                                                const int32_t* __restrict__ slot, const int32_t* __restrict__ block_table,
                                                                int max_pages, int page_size, TC* __restrict__ pool,
                                                                TC* __restrict__ q_out, long long ldqo) {
@@ -58,8 +80,9 @@ __global__ void __launch_bounds__(256) qk_norm_kv_store_kernel(const float* __re
   const int p = pos[t];
   const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
   TC* dst = pool + ((long long)page * page_size + p % page_size) * (nk + nv);
-  rms_to(q + t * ldq, nq, q_group, wq, eps, q_out + t * ldqo, red);
-  rms_to(k + t * ldk, nk, k_group, wk, eps, dst, red);
+  if (rot.cs != nullptr) rot.cs += (long long)p * rot.dims;
+  rms_to(q + t * ldq, nq, q_group, wq, eps, q_out + t * ldqo, red, rot);
+  rms_to(k + t * ldk, nk, k_group, wk, eps, dst, red, rot);
   for (int c = threadIdx.x; c < nv; c += blockDim.x) stf(dst + nk + c, v[t * ldv + c]);
 }
 
@@ -134,10 +157,11 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attn_kernel(const TQ* _
                                                                      int dv, int maps, const TC* __restrict__ pool,
                                                                      const int32_t* __restrict__ block_table, int max_pages,
                                                                      int page_size, const int32_t* __restrict__ pos,
-                                                                     const int32_t* __restrict__ slot, int window, int keep_first,
+                                                                     const int32_t* __restrict__ slot, int window, int chunk, int keep_first,
                                                                      float scale, float softcap, const float* __restrict__ dist_bias,
                                                                      const float* __restrict__ sink, const float* __restrict__ gate,
-                                                                     long long ldg, int gate_act, TY* __restrict__ out, long long ldo) {
+                                                                     long long ldg, int gate_act, int gate_heads, TY* __restrict__ out,
+                                                                     long long ldo) {
   extern __shared__ float sm[];  // q [d] | acc [warps][dv] | m [warps] | l [warps]
   // blockIdx.y = head * maps + map: queries and outputs are laid out [head][map][.], keys [key/value head][map][d]
   const int t = blockIdx.x, hm = blockIdx.y, h = hm / maps, mp = hm - h * maps, kvh = h / (H / G);
@@ -149,8 +173,8 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attn_kernel(const TQ* _
   for (int c = threadIdx.x; c < d; c += blockDim.x) sq[c] = ldf(q + (long long)t * ldq + hm * d + c);
   __syncthreads();
   const int p = pos[t];
-  const int first = max(0, p - window + 1);
-  const int kept = min(keep_first, first);   // keys 0 .. kept - 1 lie before the window and are seen all the same
+  const int first = max(max(0, p - window + 1), p - p % chunk);   // start of the window or of the row's chunk
+  const int kept = min(keep_first, first);   // keys 0 .. kept - 1 lie before it and are seen all the same
   const int32_t* bt = block_table + (long long)slot[t] * max_pages;
   const int W = G * (maps * d + dv);
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
@@ -208,7 +232,7 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attn_kernel(const TQ* _
     for (int w = 0; w < kWinWarps; ++w) o += sacc[w * dv + c] * f[w];
     o *= inv;
     if (gate != nullptr) {
-      const float z = gate[(long long)t * ldg + hm * dv + c];
+      const float z = gate[(long long)t * ldg + (gate_heads ? hm : hm * dv + c)];
       o *= gate_act == 1 ? z / (1.f + expf(-z)) : (gate_act == 2 ? 1.f / (1.f + expf(-z)) : z);
     }
     stf(out + (long long)t * ldo + hm * dv + c, o);
@@ -217,9 +241,9 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attn_kernel(const TQ* _
 
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Tensor-core kernel (bf16; head widths multiples of 16, values up to 128 wide, heads per key/value head a divisor of 64).
+// Tensor-core kernel (bf16; head widths multiples of 16, values up to 128 wide, up to 64 heads per key/value head).
 // mma.sync.m16n8k16 over 64-key tiles staged by cp.async straight out of the pages, two buffers. The 64 rows of a tile are
-// (token, query head) pairs of ONE key/value head - 64 / (H / G) consecutive tokens of one request - so the heads of a group share
+// (token, query head) pairs of ONE key/value head - up to floor(64 / (H / G)) consecutive tokens of one request - so the heads of a group share
 // the staged keys and values. Four warps of 16 rows; S = Q K^T, then scale, soft cap (tanh.approx), distance bias and window
 // mask on the accumulators, online softmax in base 2, P (bf16, from the accumulator registers) times V through ldmatrix.trans.
 // Work items: int32[4] (first_row, n_tok, slot, first_pos) from the host, or - items == NULL - every row an item of its own,
@@ -264,12 +288,12 @@ struct WinMmaArgs {
   const int32_t* slot;
   const float* bias;      // [window][H] or NULL
   const float* sink;      // [H] or NULL: one more term exp(sink[h]) in every softmax denominator
-  const float* gate;      // [T][ldg] or NULL: the output is multiplied by act(gate) elementwise
+  const float* gate;      // [T][ldg] or NULL: the output is multiplied by act(gate) elementwise, or (gate_heads) by one gate per head and map
   long long ldg;
-  int gate_act;
+  int gate_act, gate_heads;
   void* out;
   long long ldo;
-  int max_pages, page_size, H, G, d, dv, window, maps, keep_first;
+  int max_pages, page_size, H, G, d, dv, window, chunk, maps, keep_first;
   float scale, softcap;
   int q_rows;             // rows of the query tile held in shared memory: 64, or the next multiple of 16 above H / G when every item is one token
   int bias_in_smem;       // the bias columns of this key/value head's query heads are staged in shared memory ([window][H / G])
@@ -309,11 +333,13 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WinMmaArgs a) {
   const int32_t* bt = a.bt + (long long)slot * a.max_pages;
   // key ranges: the kept first keys that lie before the window of the item's first row (none when they touch the window: then
   // the window range simply starts at 0), then the window range up to the item's last row
-  int k_begin = max(0, first_pos - a.window + 1);
+  int k_begin = max(max(0, first_pos - a.window + 1), first_pos - first_pos % a.chunk);
   const int k_end = first_pos + n_tok;
   int kept_end = min(a.keep_first, k_begin);
   if (kept_end == k_begin) k_begin = 0, kept_end = 0;
   const int kept_tiles = (kept_end + kWmKeys - 1) / kWmKeys, n_tiles = kept_tiles + (k_end - k_begin + kWmKeys - 1) / kWmKeys;
+  // first key each of this thread's rows sees behind the kept ones: the start of its window or of its chunk
+  const int low0 = p0 < 0 ? 0 : max(p0 - a.window + 1, p0 - p0 % a.chunk), low1 = p1 < 0 ? 0 : max(p1 - a.window + 1, p1 - p1 % a.chunk);
   const int roww = a.G * (a.maps * d + dv);
   // two threads per key: one page lookup per thread and tile, then 16-byte copies at a constant stride
   auto stage = [&](int buf, int tile) {
@@ -380,10 +406,10 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WinMmaArgs a) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = j0 + n * 8 + 2 * t4 + (e & 1);
-          const int p = e < 2 ? p0 : p1, hh = e < 2 ? h0 : h1;
+          const int p = e < 2 ? p0 : p1, hh = e < 2 ? h0 : h1, low = e < 2 ? low0 : low1;
           const int dist = p - key;
           float v = -INFINITY;
-          if (key < j_end && dist >= 0 && (dist < a.window || key < a.keep_first)) {
+          if (key < j_end && dist >= 0 && (key >= low || key < a.keep_first)) {
             v = s[n][e] * a.scale;
             if (a.softcap > 0.f) v = a.softcap * tanh_approx(v * inv_cap);
             if (dist < a.window) {   // the table has one row per distance inside the window
@@ -456,13 +482,18 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WinMmaArgs a) {
     l0 = l0 * f0 + exp2f(s0 - r0);
     l1 = l1 * f1 + exp2f(s1 - r1);
   }
-  const float i0 = f0 / l0, i1 = f1 / l1;
+  float i0 = f0 / l0, i1 = f1 / l1;
   const long long tr0 = first_row + row0 / rep, tr1 = first_row + row1 / rep;
+  auto gact = [&](float z) { return a.gate_act == 1 ? z / (1.f + __expf(-z)) : (a.gate_act == 2 ? 1.f / (1.f + __expf(-z)) : z); };
+  const bool elem_gate = a.gate != nullptr && !a.gate_heads;
+  if (a.gate != nullptr && a.gate_heads) {
+    if (row0 < n_rows) i0 *= gact(a.gate[tr0 * a.ldg + h0 * a.maps + mp]);
+    if (row1 < n_rows) i1 *= gact(a.gate[tr1 * a.ldg + h1 * a.maps + mp]);
+  }
   TO* out0 = static_cast<TO*>(a.out) + tr0 * a.ldo + (h0 * a.maps + mp) * dv;
   TO* out1 = static_cast<TO*>(a.out) + tr1 * a.ldo + (h1 * a.maps + mp) * dv;
-  const float* g0 = a.gate != nullptr ? a.gate + tr0 * a.ldg + (h0 * a.maps + mp) * dv : nullptr;
-  const float* g1 = a.gate != nullptr ? a.gate + tr1 * a.ldg + (h1 * a.maps + mp) * dv : nullptr;
-  auto gact = [&](float z) { return a.gate_act == 1 ? z / (1.f + __expf(-z)) : (a.gate_act == 2 ? 1.f / (1.f + __expf(-z)) : z); };
+  const float* g0 = elem_gate ? a.gate + tr0 * a.ldg + (h0 * a.maps + mp) * dv : nullptr;
+  const float* g1 = elem_gate ? a.gate + tr1 * a.ldg + (h1 * a.maps + mp) * dv : nullptr;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     if (j < nv) {
@@ -760,18 +791,21 @@ extern "C" int omc_diff_heads_gate(const float* a, long long lda, int T, int H, 
 }
 
 extern "C" int omc_qk_norm_kv_store(const float* q, long long ldq, int nq, int q_group, const void* wq, const float* k, long long ldk, int nk,
-                                    int k_group, const void* wk, int w_dt, const float* v, long long ldv, int nv, float eps, int T,
+                                    int k_group, const void* wk, int w_dt, const float* v, long long ldv, int nv, float eps,
+                                    const float* cs, int head, int rot_dims, int rot_halves, int T,
                                     const int32_t* pos, const int32_t* slot, const int32_t* block_table, int max_pages, int page_size,
                                     void* pool, void* q_out, long long ldqo, int dt, void* stream) {
   if (q == nullptr || wq == nullptr || k == nullptr || wk == nullptr || v == nullptr || pos == nullptr || slot == nullptr ||
       block_table == nullptr || pool == nullptr || q_out == nullptr || T < 0 || nq <= 0 || nk <= 0 || nv <= 0 || page_size <= 0 || max_pages <= 0 ||
-      q_group < 0 || k_group < 0 || (q_group > 0 && nq % q_group) || (k_group > 0 && nk % k_group))
+      q_group < 0 || k_group < 0 || (q_group > 0 && nq % q_group) || (k_group > 0 && nk % k_group) ||
+      (cs != nullptr && (head <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > head || nq % head || nk % head || q_group % head || k_group % head)))
     return set_error(OMC_ERR_ARG, "omc_qk_norm_kv_store: bad argument");
   if (T == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const HeadRotation rot{rot_dims > 0 ? cs : nullptr, head, rot_dims, rot_halves};
   OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(dt, TC, {
     qk_norm_kv_store_kernel<TW, TC><<<T, 256, 0, st>>>(q, ldq, nq, q_group, static_cast<const TW*>(wq), k, ldk, nk, k_group, static_cast<const TW*>(wk), v,
-                                                       ldv, nv, eps, pos, slot, block_table, max_pages, page_size,
+                                                       ldv, nv, eps, rot, pos, slot, block_table, max_pages, page_size,
                                                        static_cast<TC*>(pool), static_cast<TC*>(q_out), ldqo);
   }))
   return check_launch("omc_qk_norm_kv_store");
@@ -779,10 +813,10 @@ extern "C" int omc_qk_norm_kv_store(const float* q, long long ldq, int nq, int q
 
 extern "C" int omc_window_attn(const void* q, long long ldq, int T, int H, int G, int d, int dv, int maps, const void* pool, int dt,
                                const int32_t* block_table, int max_pages, int page_size, const int32_t* pos, const int32_t* slot,
-                               int window, int keep_first, float scale, float softcap, const float* dist_bias, const float* sink,
-                               const float* gate, long long ldg, int gate_act, void* out, int out_dt, long long ldo, void* stream) {
+                               int window, int chunk, int keep_first, float scale, float softcap, const float* dist_bias, const float* sink,
+                               const float* gate, long long ldg, int gate_act, int gate_heads, void* out, int out_dt, long long ldo, void* stream) {
   if (q == nullptr || pool == nullptr || block_table == nullptr || pos == nullptr || slot == nullptr || out == nullptr || T < 0 ||
-      H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || maps < 1 || window < 1 || keep_first < 0 || page_size <= 0 || max_pages <= 0 ||
+      H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || maps < 1 || window < 1 || chunk < 1 || keep_first < 0 || page_size <= 0 || max_pages <= 0 ||
       gate_act < 0 || gate_act > 2)
     return set_error(OMC_ERR_ARG, "omc_window_attn: bad argument");
   if (T == 0) return OMC_OK;
@@ -794,8 +828,8 @@ extern "C" int omc_window_attn(const void* q, long long ldq, int T, int H, int G
   OMC_DT_SWITCH(dt, TC, OMC_DT_SWITCH(out_dt, TY, {
     window_attn_kernel<TC, TC, TY><<<dim3(T, H * maps), kWinWarps * 32, smem, st>>>(static_cast<const TC*>(q), ldq, H, G, d, dv, maps,
                                                                                    static_cast<const TC*>(pool), block_table, max_pages,
-                                                                                   page_size, pos, slot, window, keep_first, scale, softcap,
-                                                                                   dist_bias, sink, gate, ldg, gate_act, static_cast<TY*>(out), ldo);
+                                                                                   page_size, pos, slot, window, chunk, keep_first, scale, softcap,
+                                                                                   dist_bias, sink, gate, ldg, gate_act, gate_heads, static_cast<TY*>(out), ldo);
   }))
   return check_launch("omc_window_attn");
 }
@@ -803,15 +837,15 @@ extern "C" int omc_window_attn(const void* q, long long ldq, int T, int H, int G
 extern "C" int omc_window_attn_mma_ok(int H, int G, int d, int dv) {
   if (H <= 0 || G <= 0 || H % G) return 0;
   const int rep = H / G;
-  return (d % 16 == 0 && dv % 16 == 0 && d >= 16 && d <= 256 && dv >= 16 && dv <= 128 && rep <= 64 && 64 % rep == 0) ? 1 : 0;
+  return (d % 16 == 0 && dv % 16 == 0 && d >= 16 && d <= 256 && dv >= 16 && dv <= 128 && rep <= 64) ? 1 : 0;
 }
 
 extern "C" int omc_window_attn_mma(const void* q, long long ldq, int T, int H, int G, int d, int dv, int maps, const void* pool,
                                    const int32_t* block_table, int max_pages, int page_size, const int32_t* items, int n_items,
-                                   const int32_t* pos, const int32_t* slot, int window, int keep_first, float scale, float softcap,
-                                   const float* dist_bias, const float* sink, const float* gate, long long ldg, int gate_act, void* out,
+                                   const int32_t* pos, const int32_t* slot, int window, int chunk, int keep_first, float scale, float softcap,
+                                   const float* dist_bias, const float* sink, const float* gate, long long ldg, int gate_act, int gate_heads, void* out,
                                    int out_dt, long long ldo, void* stream) {
-  if (q == nullptr || pool == nullptr || block_table == nullptr || out == nullptr || T < 0 || window < 1 || maps < 1 || keep_first < 0 || page_size <= 0 ||
+  if (q == nullptr || pool == nullptr || block_table == nullptr || out == nullptr || T < 0 || window < 1 || chunk < 1 || maps < 1 || keep_first < 0 || page_size <= 0 ||
       gate_act < 0 || gate_act > 2 || max_pages <= 0 || (items == nullptr && (pos == nullptr || slot == nullptr)) || n_items < 0)
     return set_error(OMC_ERR_ARG, "omc_window_attn_mma: bad argument");
   if (!omc_window_attn_mma_ok(H, G, d, dv) || ldq % 8 || ldo % 2 || reinterpret_cast<uintptr_t>(q) % 16 || reinterpret_cast<uintptr_t>(pool) % 16)
@@ -820,7 +854,7 @@ extern "C" int omc_window_attn_mma(const void* q, long long ldq, int T, int H, i
   if (n == 0) return OMC_OK;
   if ((long long)G * maps > 65535) return set_error(OMC_ERR_SHAPE, "omc_window_attn_mma: more than 65535 key/value heads");
   WinMmaArgs a{static_cast<const bf16_t*>(q), ldq, static_cast<const bf16_t*>(pool), block_table, items, pos, slot, dist_bias, sink, gate, ldg,
-               gate_act, out, ldo, max_pages, page_size, H, G, d, dv, window, maps, keep_first, scale, softcap, kWmRows, 0};
+               gate_act, gate_heads, out, ldo, max_pages, page_size, H, G, d, dv, window, chunk, maps, keep_first, scale, softcap, kWmRows, 0};
   if (items == nullptr) a.q_rows = ((H / G + 15) / 16) * 16;   // one token per item: only H / G rows exist, and a smaller tile lets more CTAs share an SM
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   size_t smem = sizeof(bf16_t) * ((size_t)a.q_rows * (d + 8) + 2 * (size_t)kWmKeys * (d + 8) + 2 * (size_t)kWmKeys * (dv + 8));

@@ -4,8 +4,8 @@
 page by page as a request grows). `PagedLatentCache` stores, per layer, one row per token - the latent followed by the rotated
 key part - in pages of `page_size` tokens addressed through an int32 block table [slots, max_pages]; layers may differ in row
 width, so every layer has its own pool tensor over the same page ids; a layer of width 0 caches nothing and has no pool.
-`PagedStateCache` adds what mixers with a fixed-size memory need: named fp32 state tensors per layer with one entry per slot
-(recurrent matrices, the last inputs of short convolutions). Slots are handed out by the same scheduler that hands out pages.
+`PagedStateCache` adds what mixers with a fixed-size memory need: named state tensors per layer with one entry per slot (fp32
+recurrent matrices, the last inputs of short convolutions; integers such as the last token). Slots are handed out by the same scheduler that hands out pages.
 """
 from __future__ import annotations
 
@@ -76,20 +76,22 @@ class PagedLatentCache:
 
 class PagedStateCache(PagedLatentCache):
     """PagedLatentCache + states[layer][name]: fp32 [slots, *shape] for every entry of state_shapes[layer] ({} for a layer without
-    state). A request's state lives in its slot from admission to release. The kernels that carry a state start from zero when a
+    state; an entry (shape, dtype) has that dtype; entries behind the last layer belong to the model as a whole). A request's state lives in its slot from admission to release. The kernels that carry a state start from zero when a
     portion begins at position 0, so a slot needs no clearing when it changes hands; `poison_slot` overwrites a slot's states
-    with NaN, which makes any read of a previous owner's state visible (tests, debugging)."""
+    with NaN (integers: -1), which makes any read of a previous owner's state visible (tests, debugging)."""
 
     def __init__(self, widths: Sequence[int], state_shapes: Sequence[dict], n_pages: int, n_slots: int, page_size: int,
                  dtype: torch.dtype, device, max_pages_per_slot: int = 0):
         super().__init__(widths, n_pages, n_slots, page_size, dtype, device, max_pages_per_slot)
-        self.states = [{name: torch.zeros(n_slots, *shape, device=device, dtype=torch.float32) for name, shape in shapes.items()}
-                       for shapes in state_shapes]
+        def zeros(shape):
+            shape, dt = shape if len(shape) == 2 and isinstance(shape[1], torch.dtype) else (shape, torch.float32)
+            return torch.zeros(n_slots, *shape, device=device, dtype=dt)
+        self.states = [{name: zeros(shape) for name, shape in shapes.items()} for shapes in state_shapes]
 
     def poison_slot(self, slot: int):
         for layer in self.states:
             for t in layer.values():
-                t[slot].fill_(float("nan"))
+                t[slot].fill_(float("nan") if t.dtype.is_floating_point else -1)
 
     def state_bytes_per_slot(self) -> int:
-        return sum(t[0].numel() * 4 for layer in self.states for t in layer.values())
+        return sum(t[0].numel() * t.element_size() for layer in self.states for t in layer.values())

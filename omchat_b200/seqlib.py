@@ -26,6 +26,7 @@ SIGNATURES = {
     "omc_last_error": (c_char_p, []),
     "omc_linear": (_I, [_P, _I, _L, _L, _P, _I, _L, _L, _P, _I, _L, _L, _I, _I, _I, _I, _F, _I, _P, _L, _P]),
     "omc_linear_bias": (_I, [_P, _I, _L, _L, _P, _I, _L, _L, _P, _I, _L, _L, _I, _I, _I, _I, _F, _I, _P, _L, _P, _L, _P]),
+    "omc_linear_gate": (_I, [_P, _I, _L, _L, _P, _I, _L, _L, _P, _I, _L, _L, _I, _I, _I, _I, _F, _I, _P, _I, _L, _L, _P]),
     "omc_post_norm_residual": (_I, [_P, _L, _P, _P, _L, _P, _P, _I, _F, _F, _P, _L, _P, _P, _I, _L, _I, _I, _P]),
     "omc_glu_mul": (_I, [_P, _I, _L, _I, _I, _I, _F, _F, _F, _P, _I, _L, _P, _I, _P]),
     "omc_embed_sinusoid": (_I, [_P, _P, _I, _P, _I, _I, _I, _F, _P, _P, _L, _P]),
@@ -38,22 +39,25 @@ SIGNATURES = {
     "omc_pos_qkv_store": (_I, [_P, _L, _I, _P, _L, _I, _I, _P, _L, _I, _P, _I, _F, _I, _I, _F, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _P]),
     "omc_moe_combine_depth": (_I, [_P, _L, _P, _P, _I, _P, _L, _P, _L, _F, _P, _L, _F, _F, _P, _L, _L, _I, _P, _I, _P, _L, _I, _I, _P]),
     "omc_conv_qk_norm_kv_store": (_I, [_P, _L, _I, _I, _P, _I, _I, _P, _P, _P, _I, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _L, _I, _I, _P]),
-    "omc_linear_state_scan": (_I, [_P, _L, _P, _L, _P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P]),
+    "omc_linear_state_scan": (_I, [_P, _L, _P, _L, _P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P]),
     "omc_map_rows": (_I, [_P, _L, _I, _I, _I, _P, _P, _I, _F, _P]),
     "omc_gated_rms_rows": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _L, _I, _P, _I, _L, _P]),
-    "omc_qk_norm_kv_store": (_I, [_P, _L, _I, _I, _P, _P, _L, _I, _I, _P, _I, _P, _L, _I, _F, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _P]),
-    "omc_window_attn": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _F, _F, _P, _P, _P, _L, _I, _P, _I, _L, _P]),
+    "omc_gate_rms_rows": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _I, _L, _I, _P, _I, _L, _P]),
+    "omc_qk_norm_kv_store": (_I, [_P, _L, _I, _I, _P, _P, _L, _I, _I, _P, _I, _P, _L, _I, _F, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _P]),
+    "omc_window_attn": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _F, _F, _P, _P, _P, _L, _I, _I, _P, _I, _L, _P]),
     "omc_window_attn_mma_ok": (_I, [_I, _I, _I, _I]),
-    "omc_window_attn_mma": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _P, _I, _I, _F, _F, _P, _P, _P, _L, _I, _P, _I, _L, _P]),
+    "omc_window_attn_mma": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _F, _F, _P, _P, _P, _L, _I, _I, _P, _I, _L, _P]),
     "omc_diff_attn_pair_ok": (_I, [_I, _I, _I, _I]),
     "omc_diff_attn_pair": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _I, _I, _F, _F, _F, _F, _P, _L, _I, _P, _I, _L, _P]),
     "omc_ln_residual": (_I, [_P, _L, _F, _P, _L, _P, _L, _P, _P, _I, _P, _P, _I, _F, _P, _L, _P, _I, _L, _I, _I, _P]),
+    "omc_rms_residual": (_I, [_P, _L, _P, _L, _P, _L, _P, _P, _I, _P, _I, _F, _P, _L, _P, _I, _L, _I, _I, _P]),
+    "omc_embed_bigram": (_I, [_P, _P, _P, _I, _P, _I, _I, _I, _P, _I, _I, _I, _P, _P, _F, _P, _L, _P, _I, _L, _I, _P]),
     "omc_rglru_scan": (_I, [_P, _I, _L, _P, _L, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _F, _P]),
     "omc_embed_scale": (_I, [_P, _I, _P, _I, _I, _I, _F, _P, _L, _P, _I, _L, _P]),
     "omc_rms_rows": (_I, [_P, _L, _P, _I, _I, _F, _P, _I, _L, _I, _I, _P]),
     "omc_norm_residual": (_I, [_P, _L, _P, _I, _F, _P, _L, _P, _I, _L, _I, _I, _P]),
     "omc_latent_kv_store": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _I, _P, _P, _P, _I, _I, _P, _I, _P]),
-    "omc_latent_rope_store": (_I, [_P, _L, _I, _I, _I, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P, _P, _I, _L, _I, _I, _P, _P, _I, _P]),
+    "omc_latent_rope_store": (_I, [_P, _L, _I, _I, _I, _P, _F, _P, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _L, _I, _I, _P, _P, _I, _P]),
     "omc_moe_plan_scatter_small": (_I, [_P, _I, _I, _I, _P, _P, _P, _I, _L, _I, _I, _P, _I, _P, _P, _L, _P, _P]),
     "omc_rotary_q": (_I, [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P]),
     "omc_latent_attn": (_I, [_P, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _P, _I, _P, _L, _F, _P, _P]),
@@ -108,8 +112,10 @@ def _dt(t: Optional[torch.Tensor]) -> int:
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, M: Optional[int] = None, N: Optional[int] = None,
            K: Optional[int] = None, ldx: Optional[int] = None, ldw: Optional[int] = None, ldy: Optional[int] = None,
            batch: int = 1, sx: int = 0, sw: int = 0, sy: int = 0, alpha: float = 1.0, act: int = ACT_NONE,
-           tile_group: Optional[torch.Tensor] = None, group_stride: int = 0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out = act(alpha * x @ w^T (+ bias)). With the defaults x [M, K], w [N, K], out [M, N] are 2-D row-strided tensors; the keyword
+           tile_group: Optional[torch.Tensor] = None, group_stride: int = 0, bias: Optional[torch.Tensor] = None,
+           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out = act(alpha * x @ w^T (+ bias)), times sigmoid(gate) with a gate [M, batch * N] (fp32 or bf16; batch item b uses the columns
+    from b * N on). With the defaults x [M, K], w [N, K], out [M, N] are 2-D row-strided tensors; the keyword
     overrides describe batched column slices (heads) or a grouped product over expert-sorted row tiles (see the header)."""
     _need_cuda(x, w, out, tile_group)
     M = x.shape[0] if M is None else M
@@ -118,7 +124,12 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, M: Optional[i
     ldx = x.stride(0) if ldx is None else ldx
     ldw = w.stride(-2) if ldw is None else ldw
     ldy = out.stride(0) if ldy is None else ldy
-    if bias is not None:
+    if gate is not None:
+        _need_cuda(gate)
+        assert gate.stride(1) == 1 and gate.shape == (M, batch * N) and bias is None and tile_group is None
+        rc = load().omc_linear_gate(_ptr(x), _dt(x), ldx, sx, _ptr(w), _dt(w), ldw, sw, _ptr(out), _dt(out), ldy, sy, M, N, K, batch,
+                                    alpha, act, _ptr(gate), _dt(gate), gate.stride(0), N, _stream())
+    elif bias is not None:
         _need_cuda(bias)
         assert bias.dtype == w.dtype and bias.numel() == N and batch == 1
         rc = load().omc_linear_bias(_ptr(x), _dt(x), ldx, sx, _ptr(w), _dt(w), ldw, sw, _ptr(out), _dt(out), ldy, sy, M, N, K, batch,
@@ -188,16 +199,16 @@ def latent_kv_store(dkv: torch.Tensor, r: int, dr: int, w: torch.Tensor, eps: fl
 
 
 def latent_rope_store(dkv: Optional[torch.Tensor], r: int, dr: int, w, eps: float, cs, rot_dims: int, pos, slot, block_table, page_size: int, pool, q,
-                      H: int, dn: int, qcat, qn: Optional[torch.Tensor] = None):
+                      H: int, dn: int, qcat, qn: Optional[torch.Tensor] = None, rot_halves: bool = False):
     """latent_kv_store + rotary_q in one launch (w, pool, qcat of one dtype, q of that dtype or fp32). dkv None: the queries only. qn
-    [T, H * dn]: receives the unrotated query parts."""
+    [T, H * dn]: receives the unrotated query parts. rot_halves: pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)."""
     _need_cuda(dkv, w, cs, pos, slot, block_table, pool, q, qcat, qn)
     assert qcat.is_contiguous() and q.stride(1) == 1 and (qn is None or (qn.is_contiguous() and qn.dtype == qcat.dtype and qn.shape[1] == H * dn))
     if dkv is not None:
         assert dkv.dtype == torch.float32 and dkv.stride(1) == 1 and w.dtype == pool.dtype == qcat.dtype
         assert block_table.is_contiguous() and pool.is_contiguous() and pool.shape[-1] == r + dr
-    rc = load().omc_latent_rope_store(_ptr(dkv), dkv.stride(0) if dkv is not None else 0, q.shape[0], r, dr, _ptr(w), eps, _ptr(cs), rot_dims, _ptr(pos),
-                                      _ptr(slot), _ptr(block_table), block_table.shape[1], page_size, _ptr(pool), _ptr(q), _dt(q), q.stride(0), H, dn,
+    rc = load().omc_latent_rope_store(_ptr(dkv), dkv.stride(0) if dkv is not None else 0, q.shape[0], r, dr, _ptr(w), eps, _ptr(cs), rot_dims,
+                                      1 if rot_halves else 0, _ptr(pos), _ptr(slot), _ptr(block_table), block_table.shape[1], page_size, _ptr(pool), _ptr(q), _dt(q), q.stride(0), H, dn,
                                       _ptr(qcat), _ptr(qn), _dt(qcat), _stream())
     _check(rc, "omc_latent_rope_store")
 
@@ -451,6 +462,43 @@ def ln_residual(x: torch.Tensor, alpha: float, nw: torch.Tensor, nb: torch.Tenso
     return x_out if xb is None else xb
 
 
+def rms_residual(x: torch.Tensor, nw: Optional[torch.Tensor], eps: float, *, y: Optional[torch.Tensor] = None, ys: Optional[torch.Tensor] = None,
+                 slot_of: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, top: int = 0, x_out: Optional[torch.Tensor] = None,
+                 xb: Optional[torch.Tensor] = None):
+    """v = x + y + sum_j w[t, j] ys[slot_of[t, j]] (absent terms are zero) -> x_out (fp32, may be x) and / or its RMS norm with weight nw
+    -> xb (the rounded row)."""
+    _need_cuda(x, nw, y, ys, slot_of, w, x_out, xb)
+    C = x.shape[1]
+    for t in (x, y, ys, x_out):
+        assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
+    assert (xb is None or (xb.stride(1) == 1 and nw.numel() == C)) and (ys is None or (slot_of.is_contiguous() and w.is_contiguous() and w.dtype == torch.float32))
+
+    def ld(t):
+        return t.stride(0) if t is not None else 0
+    rc = load().omc_rms_residual(_ptr(x), ld(x), _ptr(y), ld(y), _ptr(ys), ld(ys), _ptr(slot_of), _ptr(w), top, _ptr(nw), _dt(nw), eps, _ptr(x_out),
+                                 ld(x_out), _ptr(xb), _dt(xb), ld(xb), x.shape[0], C, _stream())
+    _check(rc, "omc_rms_residual")
+    return x_out if xb is None else xb
+
+
+def embed_bigram(ids: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor, mul_prev: int, mul_cur: int,
+                 prev: torch.Tensor, h32: torch.Tensor, *, nw: Optional[torch.Tensor] = None, eps: float = 0.0, xb: Optional[torch.Tensor] = None,
+                 single_rows: bool = False):
+    """h32 = table[ids] + bigram[hash of (previous token, token)] (bigram has buckets + 1 rows, the last one for first tokens); prev int32
+    [slots]: the last token of every request, read and updated; xb: the rounded RMS norm of h32 with weight nw."""
+    _need_cuda(ids, pos, slot, table, bigram, prev, h32, nw, xb)
+    T, C, buckets = ids.numel(), table.shape[1], bigram.shape[0] - 1
+    assert ids.dtype == pos.dtype == slot.dtype == prev.dtype == torch.int32 and h32.dtype == torch.float32 and table.dtype == bigram.dtype
+    assert table.is_contiguous() and bigram.is_contiguous() and bigram.shape[1] == C and prev.is_contiguous()
+    assert xb is None or (nw.dtype == table.dtype and nw.numel() == C and xb.stride(1) == 1)
+    rc = load().omc_embed_bigram(_ptr(ids), _ptr(pos), _ptr(slot), T, _ptr(table), _dt(table), C, table.shape[0], _ptr(bigram), buckets,
+                                 mul_prev % buckets, mul_cur % buckets, _ptr(prev), _ptr(nw), eps, _ptr(h32), h32.stride(0), _ptr(xb), _dt(xb),
+                                 xb.stride(0) if xb is not None else 0, 1 if single_rows else 0, _stream())
+    _check(rc, "omc_embed_bigram")
+    if not single_rows:
+        _core.add_launches(1)
+
+
 def glu_mul(z: torch.Tensor, n: int, act: int, out: torch.Tensor, limit: float = 0.0, slope: float = 1.0, shift: float = 0.0,
             tile_group: Optional[torch.Tensor] = None, tile: int = 0):
     """out[:, c] = act(z[:, c]) * z[:, n + c]. ACT_CLAMP_SWISH: g = min(z[:, c], limit), u = clamp(z[:, n + c], -limit, limit),
@@ -465,7 +513,7 @@ def glu_mul(z: torch.Tensor, n: int, act: int, out: torch.Tensor, limit: float =
 
 # ---- state mixers
 GATE_NONE, GATE_SILU, GATE_SIGMOID = 0, 1, 2
-DECAY_CONST, DECAY_HEAD, DECAY_CHANNEL, DECAY_GIVEN, DECAY_SIGMOID_POW, DECAY_GIVEN_MINUS_ONE = 0, 1, 2, 3, 4, 5
+DECAY_CONST, DECAY_HEAD, DECAY_CHANNEL, DECAY_GIVEN, DECAY_SIGMOID_POW, DECAY_GIVEN_MINUS_ONE, DECAY_STEP = 0, 1, 2, 3, 4, 5, 6
 MAP_SILU, MAP_DECAY, MAP_SIGMOID_POW = 1, 2, 3
 
 
@@ -519,23 +567,28 @@ def linear_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
                       portions: int, pos: torch.Tensor, slot: torch.Tensor, H: int, G: int, dim: int, vdim: int, *, silu_in: bool = False,
                       decay_const: Optional[torch.Tensor] = None, a: Optional[torch.Tensor] = None, A_log: Optional[torch.Tensor] = None,
                       dt_bias: Optional[torch.Tensor] = None, channel_decay: bool = False, beta: Optional[torch.Tensor] = None,
-                      decay_given: bool = False, sigmoid_pow: Optional[float] = None, out_scale: float = 1.0):
+                      decay_given: bool = False, sigmoid_pow: Optional[float] = None, out_scale: float = 1.0, step_size: bool = False,
+                      D: Optional[torch.Tensor] = None):
     """The recurrence of omc_linear_state_scan; q / k / v / a / beta are fp32 2-D tensors or column slices of one.
     decay_given: `a` [T, H * dim] already holds the per-channel decays (map_rows(..., MAP_DECAY / MAP_SIGMOID_POW)).
     sigmoid_pow: the decay of key channel i is sigmoid(a[t, i] + dt_bias[i])^sigmoid_pow (with decay_given: `a` holds that decay
-    minus one). out_scale multiplies the read-out."""
-    _need_cuda(q, k, v, state, out, row_begin, pos, slot, decay_const, a, A_log, dt_bias, beta)
+    minus one). out_scale multiplies the read-out. step_size: dt = softplus(a + dt_bias) is the decay's exponent (times exp(A_log)) AND
+    what v enters the state with; D [H]: D v is added to the read-out."""
+    _need_cuda(q, k, v, state, out, row_begin, pos, slot, decay_const, a, A_log, dt_bias, beta, D)
+    assert step_size or D is None
     for t in (q, k, v, out, a, beta):
         assert t is None or (t.dtype == torch.float32 and t.stride(1) == 1)
-    for t in (decay_const, A_log, dt_bias):
+    for t in (decay_const, A_log, dt_bias, D):
         assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
     assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dim, vdim) and row_begin.dtype == torch.int32
     mode = DECAY_CONST if decay_const is not None else (DECAY_GIVEN if decay_given else (DECAY_CHANNEL if channel_decay else DECAY_HEAD))
     if sigmoid_pow is not None:   # given: by map_rows(..., MAP_SIGMOID_POW), which leaves the decay minus one
         mode = DECAY_GIVEN_MINUS_ONE if decay_given else DECAY_SIGMOID_POW
+    if step_size:
+        mode = DECAY_STEP
     rc = load().omc_linear_state_scan(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), 1 if silu_in else 0, mode,
                                       _ptr(decay_const), _ptr(a), a.stride(0) if a is not None else 0, _ptr(A_log), _ptr(dt_bias),
-                                      _ptr(beta), beta.stride(0) if beta is not None else 0, _ptr(state), _ptr(out), out.stride(0),
+                                      _ptr(D), _ptr(beta), beta.stride(0) if beta is not None else 0, _ptr(state), _ptr(out), out.stride(0),
                                       _ptr(row_begin), portions, _ptr(pos), _ptr(slot), H, G, dim, vdim,
                                       float(sigmoid_pow or 0.0), out_scale, _stream())
     _check(rc, "omc_linear_state_scan")
@@ -553,29 +606,45 @@ def gated_rms_rows(x: torch.Tensor, groups: int, n: int, w: torch.Tensor, eps: f
     return out
 
 
+def gate_rms_rows(x: torch.Tensor, groups: int, w: torch.Tensor, eps: float, gate: torch.Tensor, gate_act: int, out: torch.Tensor):
+    """v = x * act(gate); out = v / rms(v over each of `groups` equal parts of the row) * w (w as wide as the row)."""
+    _need_cuda(x, w, gate, out)
+    n = w.numel() // groups
+    assert x.dtype == torch.float32 and x.stride(1) == gate.stride(1) == out.stride(1) == 1 and w.numel() == groups * n
+    rc = load().omc_gate_rms_rows(_ptr(x), x.stride(0), x.shape[0], groups, n, _ptr(w), _dt(w), eps, _ptr(gate), _dt(gate), gate.stride(0), gate_act,
+                                  _ptr(out), _dt(out), out.stride(0), _stream())
+    _check(rc, "omc_gate_rms_rows")
+    return out
+
+
 # ---- windowed attention over a paged key/value cache
 def qk_norm_kv_store(q: torch.Tensor, wq: torch.Tensor, k: torch.Tensor, wk: torch.Tensor, v: torch.Tensor, eps: float, pos, slot,
-                     block_table: torch.Tensor, page_size: int, pool: torch.Tensor, q_out: torch.Tensor, group: int = 0):
+                     block_table: torch.Tensor, page_size: int, pool: torch.Tensor, q_out: torch.Tensor, group: int = 0, *,
+                     cs: Optional[torch.Tensor] = None, head: int = 0, rot_dims: int = 0, rot_halves: bool = False):
     """group 0: one norm over all query (key) columns, weights as wide as the projections; group > 0: one norm per `group` columns
-    with weights [group] shared by the groups (q and k are then given with their true widths)."""
-    _need_cuda(q, wq, k, wk, v, pos, slot, block_table, pool, q_out)
+    with weights [group] shared by the groups (q and k are then given with their true widths). cs fp32 [positions, rot_dims / 2, 2]
+    (cos, sin): behind the norm the first rot_dims of every `head` columns of q and k are rotated (pairs, or halves with rot_halves)."""
+    _need_cuda(q, wq, k, wk, v, pos, slot, block_table, pool, q_out, cs)
+    assert cs is None or (cs.dtype == torch.float32 and cs.is_contiguous())
     nq, nk, nv = (wq.numel(), wk.numel(), v.shape[1]) if group == 0 else (q.shape[1], k.shape[1], v.shape[1])
     assert group == 0 or (wq.numel() == group and wk.numel() == group)
     assert q.dtype == k.dtype == v.dtype == torch.float32 and q.stride(1) == k.stride(1) == v.stride(1) == 1
     assert pool.is_contiguous() and pool.shape[-1] == nk + nv and pool.dtype == q_out.dtype and wq.dtype == wk.dtype
     assert block_table.dtype == torch.int32 and block_table.is_contiguous() and q_out.stride(1) == 1
     rc = load().omc_qk_norm_kv_store(_ptr(q), q.stride(0), nq, group, _ptr(wq), _ptr(k), k.stride(0), nk, group, _ptr(wk), _dt(wq), _ptr(v), v.stride(0),
-                                     nv, eps, q.shape[0], _ptr(pos), _ptr(slot), _ptr(block_table), block_table.shape[1], page_size,
+                                     nv, eps, _ptr(cs), head, rot_dims, 1 if rot_halves else 0, q.shape[0], _ptr(pos), _ptr(slot), _ptr(block_table), block_table.shape[1], page_size,
                                      _ptr(pool), _ptr(q_out), q_out.stride(0), _dt(pool), _stream())
     _check(rc, "omc_qk_norm_kv_store")
 
 
 def window_attn(q: torch.Tensor, H: int, G: int, d: int, dv: int, pool: torch.Tensor, block_table: torch.Tensor, page_size: int, pos, slot,
                 window: int, scale: float, softcap: float, dist_bias: Optional[torch.Tensor], out: torch.Tensor, maps: int = 1,
-                keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_act: int = 0):
+                keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_act: int = 0,
+                chunk: int = WINDOW_ALL, gate_heads: bool = False):
     """q [T, H * maps * d] and pool of one dtype -> out [T, H * maps * dv]. maps: score maps per head (queries and keys of their
     own, shared values); keep_first: the first keys of a sequence stay visible behind the window; sink fp32 [H]: one more
-    denominator term exp(sink[h]); gate fp32 [T, H * maps * dv] with gate_act (GATE_*): the output is multiplied by act(gate)."""
+    denominator term exp(sink[h]); gate fp32 [T, H * maps * dv] (gate_heads: [T, H * maps], one per head) with gate_act (GATE_*): the
+    output is multiplied by act(gate). chunk: a row sees keys of its own chunk of that many positions only."""
     _need_cuda(q, pool, block_table, pos, slot, dist_bias, out, sink, gate)
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == H)
     assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
@@ -583,8 +652,8 @@ def window_attn(q: torch.Tensor, H: int, G: int, d: int, dv: int, pool: torch.Te
     assert pool.shape[-1] == G * (maps * d + dv)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous() and dist_bias.shape == (window, H))
     rc = load().omc_window_attn(_ptr(q), q.stride(0), q.shape[0], H, G, d, dv, maps, _ptr(pool), _dt(pool), _ptr(block_table),
-                                block_table.shape[1], page_size, _ptr(pos), _ptr(slot), window, keep_first, scale, softcap,
-                                _ptr(dist_bias), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, gate_act, _ptr(out),
+                                block_table.shape[1], page_size, _ptr(pos), _ptr(slot), window, chunk, keep_first, scale, softcap,
+                                _ptr(dist_bias), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, gate_act, 1 if gate_heads else 0, _ptr(out),
                                 _dt(out), out.stride(0), _stream())
     _check(rc, "omc_window_attn")
     return out
@@ -595,12 +664,21 @@ def window_attn_mma_ok(H: int, G: int, d: int, dv: int, dtype: torch.dtype) -> b
     return dtype == torch.bfloat16 and bool(load().omc_window_attn_mma_ok(H, G, d, dv))
 
 
-def window_attn_items(portions, rep: int, device) -> torch.Tensor:
+def window_attn_items(portions, rep: int, device, chunk: int = WINDOW_ALL) -> torch.Tensor:
     """Work list of omc_window_attn_mma for one step: portions [(first_row, n_rows, slot, first_pos)] cut into tiles of 64 // rep
-    tokens (rep = query heads per key/value head) -> int32 [n_items, 4] on the device."""
+    tokens (rep = query heads per key/value head) -> int32 [n_items, 4] on the device. Tiles also end where a chunk does (a tile across
+    the edge would walk the keys of both chunks), unless chunks are shorter than a key tile."""
     import numpy as np
     tok = MMA_ROWS // rep
     parts = []
+    if MMA_ROWS <= chunk < WINDOW_ALL:
+        cut = []
+        for first_row, n, slot, p0 in portions:
+            while n > 0:
+                m = min(n, chunk - p0 % chunk)
+                cut.append((first_row, m, slot, p0))
+                first_row, n, p0 = first_row + m, n - m, p0 + m
+        portions = cut
     for first_row, n, slot, p0 in portions:
         st = np.arange(0, n, tok, dtype=np.int32)
         parts.append(np.stack([first_row + st, np.minimum(tok, n - st), np.full_like(st, slot), p0 + st], axis=1))
@@ -611,8 +689,9 @@ def window_attn_items(portions, rep: int, device) -> torch.Tensor:
 def window_attn_mma(q: torch.Tensor, H: int, G: int, d: int, dv: int, pool: torch.Tensor, block_table: torch.Tensor, page_size: int,
                     items: Optional[torch.Tensor], pos, slot, window: int, scale: float, softcap: float,
                     dist_bias: Optional[torch.Tensor], out: torch.Tensor, maps: int = 1, keep_first: int = 0,
-                    sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_act: int = 0):
-    """items None: every row of q is a request of its own at (slot[t], pos[t]). maps / keep_first / sink / gate as in window_attn."""
+                    sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_act: int = 0, chunk: int = WINDOW_ALL,
+                    gate_heads: bool = False):
+    """items None: every row of q is a request of its own at (slot[t], pos[t]). maps / keep_first / sink / gate / chunk as in window_attn."""
     _need_cuda(q, pool, block_table, items, pos, slot, dist_bias, out, sink, gate)
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == H)
     assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
@@ -621,9 +700,9 @@ def window_attn_mma(q: torch.Tensor, H: int, G: int, d: int, dv: int, pool: torc
     assert items is None or (items.dtype == torch.int32 and items.is_contiguous() and items.shape[1] == 4)
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous() and dist_bias.shape == (window, H))
     rc = load().omc_window_attn_mma(_ptr(q), q.stride(0), q.shape[0], H, G, d, dv, maps, _ptr(pool), _ptr(block_table), block_table.shape[1],
-                                    page_size, _ptr(items), items.shape[0] if items is not None else 0, _ptr(pos), _ptr(slot), window,
+                                    page_size, _ptr(items), items.shape[0] if items is not None else 0, _ptr(pos), _ptr(slot), window, chunk,
                                     keep_first, scale, softcap, _ptr(dist_bias), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                    gate_act, _ptr(out), _dt(out), out.stride(0), _stream())
+                                    gate_act, 1 if gate_heads else 0, _ptr(out), _dt(out), out.stride(0), _stream())
     _check(rc, "omc_window_attn_mma")
     return out
 
