@@ -312,6 +312,10 @@ def main():
                     "this size (random weights; gated linear recurrent layers, windowed latent attention, dense and group-limited expert "
                     "feed-forwards) beside the Voduzen decoder at equal size - prefill and decode throughput and the new kernels against "
                     "their rooflines (tools/bench_munevik.py); one JSON line per size")
+    ap.add_argument("--sorupel", action="append", choices=["s", "m"], help="instead of the default workload: the Sorupel decoder at "
+                    "this size (random weights; state-space layers, latent attention, chunked attention, dense feed-forwards) beside the "
+                    "Tifisun decoder at equal size - prefill and decode throughput and the new kernels against their rooflines "
+                    "(tools/bench_sorupel.py); one JSON line per size")
     ap.add_argument("--pixel-shuffle", type=float, default=1.0, help="mm_pixel_shuffle_ratio (1.0 = reference behaviour)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -355,6 +359,14 @@ def main():
         torch.cuda.set_device(0)
         for size in args.munevik:
             print(json.dumps(measure_munevik(size, steps=max(args.steps, 8))), flush=True)
+        return
+
+    if args.sorupel:
+        import torch
+        from tools.bench_sorupel import measure as measure_sorupel
+        torch.cuda.set_device(0)
+        for size in args.sorupel:
+            print(json.dumps(measure_sorupel(size, steps=max(args.steps, 8))), flush=True)
         return
 
     import torch
