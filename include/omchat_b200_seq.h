@@ -253,12 +253,13 @@ int omc_conv_qk_norm_kv_store(const float* x, long long ldx, int T, int ch, cons
  * o_t = S^T q_t + D[head] v_t (D fp32 [H] or NULL; no beta), the decay applied as S + expm1(.) S. The read-out is multiplied by out_scale (a query scale). beta raw [T, H], squashed by a sigmoid here. silu_in: q, k, v pass silu first.
  * q / k [T, G * dim] (head h reads group h / (H / G)), v [T, H * vdim], out fp32 [T, H * vdim]. Portion i is rows
  * row_begin[i] .. row_begin[i + 1] - 1 (device int32 [portions + 1]), all of slot[row_begin[i]]; a portion whose first row has
- * position 0 starts from S = 0. Tokens are processed one after the other in every case. dim <= 256. */
+ * position 0 starts from S = 0. rows: the number of
+ * rows over all portions (how much is staged at a time depends on it). Tokens are processed one after the other in every case. dim <= 256. */
 int omc_linear_state_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, int silu_in,
                           int decay_mode, const float* decay_const, const float* a, long long lda, const float* A_log,
                           const float* dt_bias, const float* D, const float* beta, long long ldb, float* state, float* out, long long ldo,
-                          const int32_t* row_begin, int portions, const int32_t* pos, const int32_t* slot, int H, int G, int dim,
-                          int vdim, float decay_pow, float out_scale, void* stream);
+                          const int32_t* row_begin, int portions, const int32_t* pos, const int32_t* slot, int rows, int H, int G,
+                          int dim, int vdim, float decay_pow, float out_scale, void* stream);
 
 /* y[t, g * n + c] = x[t, g * n + c] / sqrt(mean_c(x[t, g * n + :]^2) + eps) * w[c] * act(gate[t, g * n + c]) for g < groups.
  * gate fp32 or NULL; gate_act 0: as is, 1: silu, 2: sigmoid. w [n] of w_dt, y of y_dt. */

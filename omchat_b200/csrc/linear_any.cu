@@ -255,7 +255,8 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
     __syncthreads();
   }
   const int g = lane >> 2, t4 = lane & 3;
-  // an accumulator pair (columns n, n + 1) goes out as one 4- or 8-byte store when the row is laid out for it
+  // an accumulator pair (columns n, n + 1) goes out as one 4- or 8-byte store when the row is laid out for it; a gate pair comes in so
+  const bool gate_pair = a.gate != nullptr && a.ldg % 2 == 0 && a.sg % 2 == 0 && reinterpret_cast<uintptr_t>(a.gate) % 8 == 0;
   const bool pair_ok = (a.ldy % 2 == 0) && (a.sy % 2 == 0) && (reinterpret_cast<uintptr_t>(a.Y) % (2 * sizeof(TY)) == 0);
 #pragma unroll
   for (int mm = 0; mm < 4; ++mm)
@@ -268,8 +269,16 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
         if (m >= a.M || n >= a.N) continue;
         const bf16_t* bias = a.bias != nullptr ? static_cast<const bf16_t*>(a.bias) + blockIdx.z * a.sbias : nullptr;
         const float b0 = bias != nullptr ? ldf(bias + n) : 0.f, b1 = (bias != nullptr && n + 1 < a.N) ? ldf(bias + n + 1) : 0.f;
-        const float v0 = gate_out(apply_act(acc[mm][nn][2 * hh] * a.alpha + b0, a.act), a, m, n);
-        const float v1 = n + 1 < a.N ? gate_out(apply_act(acc[mm][nn][2 * hh + 1] * a.alpha + b1, a.act), a, m, n + 1) : 0.f;
+        float v0 = apply_act(acc[mm][nn][2 * hh] * a.alpha + b0, a.act), v1 = apply_act(acc[mm][nn][2 * hh + 1] * a.alpha + b1, a.act);
+        if (gate_pair && n + 1 < a.N) {
+          const long long at = (long long)m * a.ldg + (long long)blockIdx.z * a.sg + n;
+          const float2 z = a.gate_dt == OMC_DT_F32 ? *reinterpret_cast<const float2*>(static_cast<const float*>(a.gate) + at)
+                                                   : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(static_cast<const bf16_t*>(a.gate) + at));
+          v0 = v0 / (1.f + __expf(-z.x)), v1 = v1 / (1.f + __expf(-z.y));
+        } else {
+          v0 = gate_out(v0, a, m, n);
+          if (n + 1 < a.N) v1 = gate_out(v1, a, m, n + 1);
+        }
         TY* dst = Y + (long long)m * a.ldy + n;
         if (pair_ok && n + 1 < a.N) {
           store_pair(dst, v0, v1);

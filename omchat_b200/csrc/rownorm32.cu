@@ -29,8 +29,9 @@ __global__ void __launch_bounds__(256) embed_bigram_kernel(const int32_t* __rest
                                                            const int32_t* __restrict__ slot, const TT* __restrict__ table, int C, int vocab,
                                                            const TT* __restrict__ bigram, int buckets, int mul_prev, int mul_cur,
                                                            int32_t* __restrict__ prev, const TT* __restrict__ nw, float eps,
-                                                           float* __restrict__ h32, long long ldh, TB* __restrict__ xb, long long ldxb, int save_here) {
-  extern __shared__ float row[];  // [C]
+                                                           float* __restrict__ h32, long long ldh, TB* __restrict__ xb, long long ldxb, int save_here, int vec) {
+  extern __shared__ __align__(16) float erow[];  // [C]
+  float* row = erow;
   __shared__ float red[33];
   __shared__ int s_row;
   const int t = blockIdx.x, id = ids[t];
@@ -49,6 +50,28 @@ __global__ void __launch_bounds__(256) embed_bigram_kernel(const int32_t* __rest
   const bool ok = id >= 0 && id < vocab;
   const TT* br = bigram + (long long)s_row * C;
   float ss = 0.f;
+  if (vec) {   // four neighbouring columns at a time
+    for (int c = threadIdx.x * 4; c < C; c += blockDim.x * 4) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f}, b[4];
+      if (ok) ld4(table + (long long)id * C + c, v);
+      ld4(br + c, b);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] += b[e], ss = fmaf(v[e], v[e], ss);
+      st4(h32 + (long long)t * ldh + c, v);
+      st4(row + c, v);
+    }
+    if (xb == nullptr) return;
+    ss = block_sum(ss, red);
+    const float rstd = 1.f / sqrtf(ss / (float)C + eps);
+    for (int c = threadIdx.x * 4; c < C; c += blockDim.x * 4) {
+      float v[4], w[4];
+      ld4(row + c, v);
+      ld4(nw + c, w);
+      const float o[4] = {v[0] * rstd * w[0], v[1] * rstd * w[1], v[2] * rstd * w[2], v[3] * rstd * w[3]};
+      st4(xb + (long long)t * ldxb + c, o);
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < C; c += blockDim.x) {
     const float v = (ok ? ldf(table + (long long)id * C + c) : 0.f) + ldf(br + c);
     h32[(long long)t * ldh + c] = v;
@@ -572,6 +595,8 @@ extern "C" int omc_embed_bigram(const int32_t* ids, const int32_t* pos, const in
   if (T == 0) return OMC_OK;
   const size_t smem = (size_t)C * sizeof(float);
   if (smem > 200 * 1024) return set_error(OMC_ERR_SHAPE, "omc_embed_bigram: row too wide for shared memory");
+  auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const int vec = C % 4 == 0 && ldh % 4 == 0 && ldxb % 4 == 0 && al16(table) && al16(bigram) && al16(nw) && al16(h32) && al16(xb) ? 1 : 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   OMC_DT_SWITCH(t_dt, TT, OMC_DT_SWITCH(xb_dt, TB, {
     if (smem > 48 * 1024) {
@@ -580,7 +605,7 @@ extern "C" int omc_embed_bigram(const int32_t* ids, const int32_t* pos, const in
     }
     embed_bigram_kernel<TT, TB><<<T, 256, smem, st>>>(ids, pos, slot, static_cast<const TT*>(table), C, vocab, static_cast<const TT*>(bigram), buckets,
                                                       mul_prev, mul_cur, prev, static_cast<const TT*>(nw), eps, h32, ldh, static_cast<TB*>(xb), ldxb,
-                                                      single_rows);
+                                                      single_rows, vec);
   }))
   if (!single_rows) last_token_save_kernel<<<(T + 255) / 256, 256, 0, st>>>(ids, slot, T, prev);
   return check_launch("omc_embed_bigram");

@@ -308,15 +308,18 @@ __device__ __forceinline__ int scan_place(int i) { return (i / DPT) * (DPT + 4) 
 // after arrival one pass turns them in place into what the recurrence uses (silu, decays, sigmoid). VEC: 16-byte copies
 // (every row starts on a 16-byte boundary and the widths are multiples of four), else 4-byte copies.
 // KIND: what enters the state - v itself, the delta rule's correction, or dt v (decay mode 6).
+// TOK: tokens per stage - kScanTok, or 1 for steps of one-token portions, whose CTAs then need little shared memory (more of them share
+// an SM and keep state loads in flight); any TOK is right for any portion.
 enum { kScanPlain = 0, kScanDelta = 1, kScanStep = 2 };
-template <int DPT, bool VEC, int KIND>
+template <int DPT, bool VEC, int KIND, int TOK>
 __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_kernel(ScanArgs a) {
   extern __shared__ __align__(16) float sm[];
   constexpr int PITCH = kScanLanes * (DPT + 4);
   const int dim = a.dim;
   const bool chan = KIND != kScanStep && a.decay_mode >= 2;   // one decay per key channel: computed here (2, 4) or given (3, 5)
   const bool minus1 = KIND == kScanStep || a.decay_mode >= 4;  // the staged value is the decay minus one
-  const int stage_floats = kScanTok * PITCH * (chan ? 3 : 2) + kScanTok * kScanCols + 2 * kScanTok;
+  constexpr int HEADW = TOK < 4 ? 4 : TOK;   // one number per token, in whole 16-byte pieces
+  const int stage_floats = TOK * PITCH * (chan ? 3 : 2) + TOK * kScanCols + 2 * HEADW;
   const int h = blockIdx.y, kvh = h / (a.H / a.G);
   const int col0 = blockIdx.x * kScanCols;
   const int r0 = a.row_begin[blockIdx.z], r1 = a.row_begin[blockIdx.z + 1];
@@ -347,10 +350,10 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
 
   auto issue = [&](int c0, int n, int stage) {
     float* sk = sm + stage * stage_floats;
-    float* sq = sk + kScanTok * PITCH;
-    float* sg = sq + kScanTok * PITCH;                       // [tok][PITCH] (per channel) or [tok]
-    float* sv = sg + (chan ? kScanTok * PITCH : kScanTok);
-    float* sb = sv + kScanTok * kScanCols;
+    float* sq = sk + TOK * PITCH;
+    float* sg = sq + TOK * PITCH;                       // [tok][PITCH] (per channel) or [tok]
+    float* sv = sg + (chan ? TOK * PITCH : HEADW);
+    float* sb = sv + TOK * kScanCols;
     if (VEC) {
       const int d4 = dim >> 2;
       for (int e = tid; e < n * d4; e += blockDim.x) {
@@ -382,22 +385,22 @@ __global__ void __launch_bounds__(kScanCols / 2 * kScanLanes) linear_state_scan_
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
 
-  issue(r0, min(kScanTok, r1 - r0), 0);
+  issue(r0, min(TOK, r1 - r0), 0);
   int stage = 0;
-  for (int c0 = r0; c0 < r1; c0 += kScanTok, stage ^= 1) {
-    const int n = min(kScanTok, r1 - c0);
-    if (c0 + kScanTok < r1) {
-      issue(c0 + kScanTok, min(kScanTok, r1 - c0 - kScanTok), stage ^ 1);
+  for (int c0 = r0; c0 < r1; c0 += TOK, stage ^= 1) {
+    const int n = min(TOK, r1 - c0);
+    if (c0 + TOK < r1) {
+      issue(c0 + TOK, min(TOK, r1 - c0 - TOK), stage ^ 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
     float* sk = sm + stage * stage_floats;
-    float* sq = sk + kScanTok * PITCH;
-    float* sg = sq + kScanTok * PITCH;
-    float* sv = sg + (chan ? kScanTok * PITCH : kScanTok);
-    float* sb = sv + kScanTok * kScanCols;
+    float* sq = sk + TOK * PITCH;
+    float* sg = sq + TOK * PITCH;
+    float* sv = sg + (chan ? TOK * PITCH : HEADW);
+    float* sb = sv + TOK * kScanCols;
     // raw inputs -> what the recurrence uses
     if (a.silu_in || a.decay_mode == 2 || a.decay_mode == 4) {
       for (int e = tid; e < n * dim; e += blockDim.x) {
@@ -1100,7 +1103,7 @@ extern "C" int omc_linear_state_scan(const float* q, long long ldq, const float*
                                      int silu_in, int decay_mode, const float* decay_const, const float* a, long long lda,
                                      const float* A_log, const float* dt_bias, const float* D, const float* beta, long long ldb, float* state,
                                      float* out, long long ldo, const int32_t* row_begin, int portions, const int32_t* pos,
-                                     const int32_t* slot, int H, int G, int dim, int vdim, float decay_pow, float out_scale, void* stream) {
+                                     const int32_t* slot, int rows, int H, int G, int dim, int vdim, float decay_pow, float out_scale, void* stream) {
   if (q == nullptr || k == nullptr || v == nullptr || state == nullptr || out == nullptr || row_begin == nullptr || pos == nullptr ||
       slot == nullptr || portions < 0 || H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || decay_mode < 0 || decay_mode > 6 ||
       (decay_mode == 0 && decay_const == nullptr) || (decay_mode != 0 && a == nullptr) || (decay_mode == 6 && beta != nullptr) || (D != nullptr && decay_mode != 6) ||
@@ -1114,32 +1117,35 @@ extern "C" int omc_linear_state_scan(const float* q, long long ldq, const float*
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int dpt = dim <= 32 ? 4 : (dim <= 64 ? 8 : (dim <= 128 ? 16 : 32));   // key channels per thread: dim / 8 lanes, rounded up to a float4
   const bool chan = decay_mode >= 2 && decay_mode <= 5;
-  const size_t stage_floats = (size_t)kScanTok * kScanLanes * (dpt + 4) * (chan ? 3 : 2) + kScanTok * kScanCols + 2 * kScanTok;
-  const size_t smem = 2 * stage_floats * sizeof(float);
-  dim3 grid((vdim + kScanCols - 1) / kScanCols, H, portions);
-  const int threads = kScanCols / 2 * kScanLanes;
   auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const bool vec = dim % 4 == 0 && vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && al16(q) && al16(k) && al16(v) &&
                    (!chan || (lda % 4 == 0 && al16(a)));
-#define OMC_SCAN_LAUNCH(DPT, VEC, KIND)                                                                                        \
-  do {                                                                                                                         \
-    static bool attr_done[kMaxDevices] = {};                                                                                   \
-    if (!attr_done[cur_device()]) {                                                                                            \
-      cudaFuncSetAttribute(linear_state_scan_kernel<DPT, VEC, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024); \
-      attr_done[cur_device()] = true;                                                                                          \
-    }                                                                                                                          \
-    linear_state_scan_kernel<DPT, VEC, KIND><<<grid, threads, smem, st>>>(s);                                                  \
+  const bool one = vec && rows <= portions;   // every portion is one token
+  const int tok = one ? 1 : kScanTok;
+  const size_t stage_floats = (size_t)tok * kScanLanes * (dpt + 4) * (chan ? 3 : 2) + tok * kScanCols + 2 * (tok < 4 ? 4 : tok);
+  const size_t smem = 2 * stage_floats * sizeof(float);
+  dim3 grid((vdim + kScanCols - 1) / kScanCols, H, portions);
+  const int threads = kScanCols / 2 * kScanLanes;
+#define OMC_SCAN_LAUNCH(DPT, VEC, KIND, TOK)                                                                                        \
+  do {                                                                                                                              \
+    static bool attr_done[kMaxDevices] = {};                                                                                        \
+    if (!attr_done[cur_device()]) {                                                                                                 \
+      cudaFuncSetAttribute(linear_state_scan_kernel<DPT, VEC, KIND, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024); \
+      attr_done[cur_device()] = true;                                                                                               \
+    }                                                                                                                               \
+    linear_state_scan_kernel<DPT, VEC, KIND, TOK><<<grid, threads, smem, st>>>(s);                                                  \
   } while (0)
-#define OMC_SCAN_KIND(DPT, VEC)                                         \
-  do {                                                                  \
-    if (decay_mode == 6) OMC_SCAN_LAUNCH(DPT, VEC, kScanStep);          \
-    else if (beta != nullptr) OMC_SCAN_LAUNCH(DPT, VEC, kScanDelta);    \
-    else OMC_SCAN_LAUNCH(DPT, VEC, kScanPlain);                         \
+#define OMC_SCAN_KIND(DPT, VEC, TOK)                                         \
+  do {                                                                       \
+    if (decay_mode == 6) OMC_SCAN_LAUNCH(DPT, VEC, kScanStep, TOK);          \
+    else if (beta != nullptr) OMC_SCAN_LAUNCH(DPT, VEC, kScanDelta, TOK);    \
+    else OMC_SCAN_LAUNCH(DPT, VEC, kScanPlain, TOK);                         \
   } while (0)
-#define OMC_SCAN_DPT(DPT)              \
-  do {                                 \
-    if (vec) OMC_SCAN_KIND(DPT, true); \
-    else OMC_SCAN_KIND(DPT, false);    \
+#define OMC_SCAN_DPT(DPT)                             \
+  do {                                                \
+    if (one) OMC_SCAN_KIND(DPT, true, 1);             \
+    else if (vec) OMC_SCAN_KIND(DPT, true, kScanTok); \
+    else OMC_SCAN_KIND(DPT, false, kScanTok);         \
   } while (0)
   if (dpt == 4) OMC_SCAN_DPT(4);
   else if (dpt == 8) OMC_SCAN_DPT(8);

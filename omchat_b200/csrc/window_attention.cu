@@ -43,11 +43,65 @@ __device__ __forceinline__ float norm_rot_value(const float* __restrict__ x, con
   return second ? v * co + o * si : v * co - o * si;
 }
 
-// One CTA per row. q: RMS norm with a plain weight (and rotation) -> q_out; k likewise -> page; v copied -> page. group 0: one norm over
-// all columns, weight [n]; group > 0: one norm per `group` consecutive columns (a warp each), weight [group] shared by the groups.
-template <typename TW, typename TD>
+// The same for four neighbouring columns (c, heads, rotated parts and their halves multiples of four).
+template <typename TW>
+__device__ __forceinline__ void norm_rot_value4(const float* __restrict__ x, const TW* __restrict__ w, int c, float rstd, const HeadRotation& rot, float (&o)[4]) {
+  float xv[4], wv[4];
+  ld4(x + c, xv);
+  ld4(w + c, wv);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) o[e] = xv[e] * rstd * wv[e];
+  if (rot.cs == nullptr) return;
+  const int i = c % rot.width;
+  if (i >= rot.dims) return;
+  if (rot.halves) {
+    const int half = rot.dims >> 1;
+    const bool second = i >= half;
+    const int f = second ? i - half : i, to = second ? -half : half;
+    float xo[4], wo[4], ca[4], cb[4];
+    ld4(x + c + to, xo);
+    ld4(w + c + to, wo);
+    ld4(rot.cs + 2 * f, ca);
+    ld4(rot.cs + 2 * f + 4, cb);
+    const float co[4] = {ca[0], ca[2], cb[0], cb[2]}, si[4] = {ca[1], ca[3], cb[1], cb[3]};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float p = xo[e] * rstd * wo[e];
+      o[e] = second ? o[e] * co[e] + p * si[e] : o[e] * co[e] - p * si[e];
+    }
+  } else {
+    float cv[4];
+    ld4(rot.cs + i, cv);   // (cos, sin) of the pairs (i, i + 1) and (i + 2, i + 3)
+#pragma unroll
+    for (int e = 0; e < 4; e += 2) {
+      const float u = o[e], v = o[e + 1];
+      o[e] = u * cv[e] - v * cv[e + 1];
+      o[e + 1] = v * cv[e] + u * cv[e + 1];
+    }
+  }
+}
+
+// q: RMS norm with a plain weight (and rotation) -> q_out; k likewise -> page; v copied -> page. group 0: one norm over all columns,
+// weight [n]; group > 0: one norm per `group` consecutive columns (a warp each), weight [group] shared by the groups.
+template <bool VEC, typename TW, typename TD>
 __device__ __forceinline__ void rms_to(const float* __restrict__ x, int n, int group, const TW* __restrict__ w, float eps,
                                        TD* __restrict__ dst, float* red, const HeadRotation& rot) {
+  if (VEC && group <= 0) {
+    float ss = 0.f;
+    for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+      float v[4];
+      ld4(x + c, v);
+      ss = fmaf(v[0], v[0], ss), ss = fmaf(v[1], v[1], ss), ss = fmaf(v[2], v[2], ss), ss = fmaf(v[3], v[3], ss);
+    }
+    ss = block_sum(ss, red);
+    const float rstd = 1.f / sqrtf(ss / (float)n + eps);
+    for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+      float o[4];
+      norm_rot_value4(x, w, c, rstd, rot, o);
+      st4(dst + c, o);
+    }
+    return;
+  }
   if (group <= 0) {
     float ss = 0.f;
     for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
@@ -67,7 +121,8 @@ __device__ __forceinline__ void rms_to(const float* __restrict__ x, int n, int g
   }
 }
 
-template <typename TW, typename TC>
+// One CTA per row for the queries (blockIdx.y 0), another for keys and values (blockIdx.y 1).
+template <typename TW, typename TC, bool VEC>
 __global__ void __launch_bounds__(256) qk_norm_kv_store_kernel(const float* __restrict__ q, long long ldq, int nq, int q_group,
                                                                const TW* __restrict__ wq, const float* __restrict__ k, long long ldk,
                                                                int nk, int k_group, const TW* __restrict__ wk, const float* __restrict__ v,
@@ -78,11 +133,14 @@ __global__ void __launch_bounds__(256) qk_norm_kv_store_kernel(const float* __re
   __shared__ float red[33];
   const long long t = blockIdx.x;
   const int p = pos[t];
+  if (rot.cs != nullptr) rot.cs += (long long)p * rot.dims;
+  if (blockIdx.y == 0) {
+    rms_to<VEC>(q + t * ldq, nq, q_group, wq, eps, q_out + t * ldqo, red, rot);
+    return;
+  }
   const int page = block_table[(long long)slot[t] * max_pages + p / page_size];
   TC* dst = pool + ((long long)page * page_size + p % page_size) * (nk + nv);
-  if (rot.cs != nullptr) rot.cs += (long long)p * rot.dims;
-  rms_to(q + t * ldq, nq, q_group, wq, eps, q_out + t * ldqo, red, rot);
-  rms_to(k + t * ldk, nk, k_group, wk, eps, dst, red, rot);
+  rms_to<VEC>(k + t * ldk, nk, k_group, wk, eps, dst, red, rot);
   for (int c = threadIdx.x; c < nv; c += blockDim.x) stf(dst + nk + c, v[t * ldv + c]);
 }
 
@@ -803,10 +861,16 @@ extern "C" int omc_qk_norm_kv_store(const float* q, long long ldq, int nq, int q
   if (T == 0) return OMC_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const HeadRotation rot{rot_dims > 0 ? cs : nullptr, head, rot_dims, rot_halves};
+  auto al16 = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
+  const bool vec = nq % 4 == 0 && nk % 4 == 0 && nv % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldqo % 4 == 0 && al16(q) && al16(k) && al16(wq) && al16(wk) &&
+                   al16(pool) && al16(q_out) && (rot.cs == nullptr || (al16(cs) && head % 4 == 0 && rot_dims % (rot_halves ? 8 : 4) == 0));
   OMC_DT_SWITCH(w_dt, TW, OMC_DT_SWITCH(dt, TC, {
-    qk_norm_kv_store_kernel<TW, TC><<<T, 256, 0, st>>>(q, ldq, nq, q_group, static_cast<const TW*>(wq), k, ldk, nk, k_group, static_cast<const TW*>(wk), v,
-                                                       ldv, nv, eps, rot, pos, slot, block_table, max_pages, page_size,
-                                                       static_cast<TC*>(pool), static_cast<TC*>(q_out), ldqo);
+    auto go = [&](auto kernel) {
+      kernel<<<dim3(T, 2), 256, 0, st>>>(q, ldq, nq, q_group, static_cast<const TW*>(wq), k, ldk, nk, k_group, static_cast<const TW*>(wk), v, ldv, nv, eps, rot,
+                                         pos, slot, block_table, max_pages, page_size, static_cast<TC*>(pool), static_cast<TC*>(q_out), ldqo);
+    };
+    if (vec) go(qk_norm_kv_store_kernel<TW, TC, true>);
+    else go(qk_norm_kv_store_kernel<TW, TC, false>);
   }))
   return check_launch("omc_qk_norm_kv_store");
 }

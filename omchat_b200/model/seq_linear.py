@@ -1,4 +1,4 @@
-"""The linear layer of the sequence-step decoders (Voduzen, Tifisun, Fofisun, Vefunex, Munevik): which kernel multiplies which matrix.
+"""The linear layer of the sequence-step decoders (Voduzen, Tifisun, Fofisun, Vefunex, Munevik, Sorupel): which kernel multiplies which matrix.
 
 Matrices with at least TENSOR_GEMM_MIN_WEIGHT elements go through the tcgen05 GEMM of the core library when the operands are bf16
 and the dimensions are multiples of 8; below it a launch is latency-bound either way and the kernel of the sequence-step library

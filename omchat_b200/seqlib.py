@@ -39,7 +39,7 @@ SIGNATURES = {
     "omc_pos_qkv_store": (_I, [_P, _L, _I, _P, _L, _I, _I, _P, _L, _I, _P, _I, _F, _I, _I, _F, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _P]),
     "omc_moe_combine_depth": (_I, [_P, _L, _P, _P, _I, _P, _L, _P, _L, _F, _P, _L, _F, _F, _P, _L, _L, _I, _P, _I, _P, _L, _I, _I, _P]),
     "omc_conv_qk_norm_kv_store": (_I, [_P, _L, _I, _I, _P, _I, _I, _P, _P, _P, _I, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _L, _I, _I, _P]),
-    "omc_linear_state_scan": (_I, [_P, _L, _P, _L, _P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P]),
+    "omc_linear_state_scan": (_I, [_P, _L, _P, _L, _P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P]),
     "omc_map_rows": (_I, [_P, _L, _I, _I, _I, _P, _P, _I, _F, _P]),
     "omc_gated_rms_rows": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _L, _I, _P, _I, _L, _P]),
     "omc_gate_rms_rows": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _I, _L, _I, _P, _I, _L, _P]),
@@ -589,7 +589,7 @@ def linear_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
     rc = load().omc_linear_state_scan(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), 1 if silu_in else 0, mode,
                                       _ptr(decay_const), _ptr(a), a.stride(0) if a is not None else 0, _ptr(A_log), _ptr(dt_bias),
                                       _ptr(D), _ptr(beta), beta.stride(0) if beta is not None else 0, _ptr(state), _ptr(out), out.stride(0),
-                                      _ptr(row_begin), portions, _ptr(pos), _ptr(slot), H, G, dim, vdim,
+                                      _ptr(row_begin), portions, _ptr(pos), _ptr(slot), q.shape[0], H, G, dim, vdim,
                                       float(sigmoid_pow or 0.0), out_scale, _stream())
     _check(rc, "omc_linear_state_scan")
     return out

@@ -357,9 +357,9 @@ def test_a_latent_row_far_back_is_found_behind_a_sink(kind):
 # --------------------------------------------------------------------------------------------------------------- recurrence
 @pytest.mark.parametrize("H,G,N,P", [(6, 3, 12, 10), (4, 1, 7, 9), (1, 1, 1, 1), (8, 2, 64, 64), (4, 4, 128, 32), (2, 1, 200, 70), (3, 3, 32, 33)])
 def test_state_space_recurrence_in_portions_over_poisoned_slots(H, G, N, P):
-    """Two requests in interleaved portions of 1 to 40 tokens; inputs are column slices of one row as in the model."""
+    """Two requests in interleaved portions of 1 to 40 tokens (once one token each); inputs are column slices of one row as in the model."""
     n = [73, 60]
-    cuts = ([0, 1, 3, 4, 40, n[0]], [0, 2, 3, 19, 20, n[1]])
+    cuts = ([0, 1, 3, 4, 5, 40, n[0]], [0, 2, 3, 19, 20, 21, n[1]])
     inner, gn = H * P, G * N
     u, dt_raw = [rand(k, inner + 2 * gn, seed=k) for k in n], [rand(k, H, seed=k + 1) for k in n]
     A_log, dt_bias, D = rand(H, seed=1, s=1.5), rand(H, seed=2) - 1.0, rand(H, seed=3)
@@ -367,7 +367,7 @@ def test_state_space_recurrence_in_portions_over_poisoned_slots(H, G, N, P):
     for use_d in (True, False):
         want = [O.ssd_recurrence(u[r][:, :inner].view(-1, H, P), u[r][:, inner:inner + gn].view(-1, G, N), u[r][:, inner + gn:].view(-1, G, N),
                                  O.softplus(dt_raw[r] + dt_bias), A_log, D if use_d else D * 0).reshape(-1, inner) for r in range(2)]
-        for step in range(5):
+        for step in range(6):
             rows, pos, slot = _cut_rows(cuts, step, (3, 1))
             ud = _dev(torch.cat([u[r][lo:hi] for r, lo, hi, _ in rows]))
             a = _dev(torch.cat([torch.cat([rand(hi - lo, 5, seed=9), dt_raw[r][lo:hi]], 1) for r, lo, hi, _ in rows]))
